@@ -13,45 +13,12 @@
 
 #include "nb_common.cuh"
 #include "nb_host.h"
+#include "nb_launch.cuh"
+#include "../../include/nativebit_b200_layered.h"
 
 namespace nb {
 
 namespace cg = cooperative_groups;
-
-// Every kernel of the decode chain is launched with programmatic stream serialization: it may be
-// scheduled while its predecessor still runs and waits for the predecessor's results before it
-// touches memory.  It releases its own successor only AFTER that wait: a successor may then read,
-// ahead of its own wait, anything written two or more launches back (the attention kernel does).
-__device__ __forceinline__ void pdl_enter() {
-  asm volatile("griddepcontrol.wait;" ::: "memory");
-  asm volatile("griddepcontrol.launch_dependents;");
-}
-
-template <typename... KArgs, typename... Args>
-static int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = grid;
-  cfg.blockDim = block;
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = st;
-  cudaLaunchAttribute attr[1];
-  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[0].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = 1;
-  return record_cuda_error(cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...));
-}
-
-__device__ __forceinline__ float warp_sum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-__device__ __forceinline__ float warp_max(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
-  return v;
-}
 
 // x[b] += delta[b] (if delta); out[b] = x[b] / sqrt(mean(x[b]^2) + eps) * w.  One CTA per row; the
 // row lives in registers (up to 16 elements per thread), so global memory is read exactly once.
@@ -647,7 +614,7 @@ __global__ void embed_rows_kernel(const __nv_bfloat16* __restrict__ table, const
 
 // The end of a decode step for one sequence per CTA: logits_out[b, v] = cap * tanh(float(logits[b, v]) / cap),
 // token[b] = index of the largest capped logit (the lowest index among equals), and CTA 0 advances the
-// position.  logits are bf16 (the LM-head product) or fp32.
+// position.  logits are bf16 (the LM-head product) or fp32.  Without logits_out: the arg-max of the logits as they are.
 constexpr int kFinishThreads = 1024;
 __global__ void __launch_bounds__(kFinishThreads) softcap_argmax_kernel(const void* __restrict__ logits, int is_bf16, int V, float cap,
                                                                         float* __restrict__ logits_out, long long* __restrict__ token,
@@ -672,8 +639,8 @@ __global__ void __launch_bounds__(kFinishThreads) softcap_argmax_kernel(const vo
     for (int j = 0; j < 8; ++j) {
       const int i = i0 + j * kFinishThreads;
       if (i < V) {
-        const float y = cap * tanhf(x[j] / cap);
-        logits_out[(size_t)b * V + i] = y;
+        const float y = logits_out ? cap * tanhf(x[j] / cap) : x[j];
+        if (logits_out) logits_out[(size_t)b * V + i] = y;
         if (y > best || (y == best && i < best_i)) { best = y; best_i = i; }   // NaN never wins, as in a max-reduction that skips it
       }
     }
@@ -720,6 +687,13 @@ extern "C" int nb_softcap_argmax(const void* logits, int logits_dtype, int B, in
   return launch_pdl(softcap_argmax_kernel, dim3(B), dim3(kFinishThreads), 0, (cudaStream_t)stream, logits,
                     logits_dtype == NB_BF16 ? 1 : 0, V, cap, logits_out, reinterpret_cast<long long*>(token),
                     reinterpret_cast<long long*>(pos));
+}
+
+extern "C" int nb_argmax(const float* logits, int B, int V, int64_t* token, int64_t* pos, void* stream) {
+  if (!logits || !token || B < 1 || V < 1) return NB_ERR_ARG;
+  if (int rc = check_device()) return rc;
+  return launch_pdl(softcap_argmax_kernel, dim3(B), dim3(kFinishThreads), 0, (cudaStream_t)stream, (const void*)logits, 0, V, 1.0f,
+                    (float*)nullptr, reinterpret_cast<long long*>(token), reinterpret_cast<long long*>(pos));
 }
 
 extern "C" int nb_add_rmsnorm(float* x, const float* delta, const float* w, float eps, float* out, int B, int C, void* stream) {

@@ -1,0 +1,304 @@
+// Dense pieces of the layered decoders: embedding lookup with a scale, the residual chain (norm after a sublayer, add,
+// norm before the next), the fp32 matrix product, and the decode matvec over bf16 weights with the chain folded in.
+#include <cuda_runtime.h>
+#include <cuda_bf16.h>
+
+#include <algorithm>
+
+#include "nb_layered.cuh"
+
+namespace nb {
+
+__global__ void __launch_bounds__(256) embed_scaled_kernel(const bf16* __restrict__ table, const long long* __restrict__ token,
+                                                           float* __restrict__ x, int V, int C, float scale) {
+  pdl_enter();
+  long long t = token[blockIdx.x];
+  t = t < 0 ? 0 : (t >= V ? V - 1 : t);
+  const bf16* row = table + (size_t)t * C;
+  for (int i = threadIdx.x; i < C; i += 256) x[(size_t)blockIdx.x * C + i] = __bfloat162float(row[i]) * scale;
+}
+
+// One CTA per row; the row stays in shared memory between the passes (a thread rereads only what it wrote).
+constexpr int kChainThreads = 256, kChainWarps = kChainThreads / 32;
+
+template <typename TH>
+__global__ void __launch_bounds__(kChainThreads) residual_norm_kernel(float* __restrict__ x, const float* __restrict__ y,
+                                                                      const float* __restrict__ wy, const float* __restrict__ w, int kind,
+                                                                      float eps, TH* __restrict__ h, int ldh, int C) {
+  extern __shared__ __align__(16) float row_s[];
+  __shared__ float red[4 * kChainWarps];
+  pdl_enter();
+  float* xr = x + (size_t)blockIdx.x * C;
+  const int tid = threadIdx.x;
+  auto each = [&](auto f) {
+    for (int i = tid; i < C; i += kChainThreads) f(row_s[i]);
+  };
+  float mean, inv;
+  if (y) {
+    const float* yr = y + (size_t)blockIdx.x * C;
+    for (int i = tid; i < C; i += kChainThreads) row_s[i] = yr[i];
+    norm_stats<kChainWarps>(kind, C, eps, red, each, mean, inv);
+    for (int i = tid; i < C; i += kChainThreads) {
+      const float v = xr[i] + (row_s[i] - mean) * inv * wy[i];
+      xr[i] = v;
+      row_s[i] = v;
+    }
+  } else {
+    for (int i = tid; i < C; i += kChainThreads) row_s[i] = xr[i];
+  }
+  if (h) {
+    norm_stats<kChainWarps>(kind, C, eps, red + 2 * kChainWarps, each, mean, inv);
+    TH* hr = h + (size_t)blockIdx.x * ldh;
+    for (int i = tid; i < C; i += kChainThreads) hr[i] = from_f<TH>((row_s[i] - mean) * inv * w[i]);
+  }
+}
+
+// ---- fp32 product: 64 x 64 output tile per CTA, 16 x 16 threads with 4 x 4 outputs each, k in steps of 16.
+constexpr int kFT = 64, kFKS = 16;
+
+__global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ x, int ldx, const bf16* __restrict__ w, int ldw,
+                                                         const float* __restrict__ bias, int act, int M, int N, int K, float* __restrict__ y,
+                                                         int ldy) {
+  __shared__ float xs[kFKS][kFT + 4], ws[kFKS][kFT + 4];
+  const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const int m0 = blockIdx.y * kFT, n0 = blockIdx.x * kFT;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kFKS) {
+    for (int i = tid; i < kFT * kFKS; i += 256) {
+      const int r = i / kFKS, k = i % kFKS;
+      xs[k][r] = (m0 + r < M && k0 + k < K) ? x[(size_t)(m0 + r) * ldx + k0 + k] : 0.f;
+      ws[k][r] = (n0 + r < N && k0 + k < K) ? __bfloat162float(w[(size_t)(n0 + r) * ldw + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kFKS; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&xs[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&ws[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+  const int n = n0 + tx * 4;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= M) continue;
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = acc[i][j] + ((bias && n + j < N) ? bias[n + j] : 0.f);
+    if (act == NB_ACT_SWIGLU_PAIRS) {
+#pragma unroll
+      for (int j = 0; j < 4; j += 2)
+        if (n + j + 1 < N) y[(size_t)m * ldy + ((n + j) >> 1)] = silu_f(v[j]) * v[j + 1];
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (n + j < N) y[(size_t)m * ldy + n + j] = v[j];
+    }
+  }
+}
+
+// ---- decode matvec.  A CTA owns a contiguous range of rows; the range, cut into items of one row x 256 columns (512
+// bytes, 16 per lane), is dealt to the CTA's warps in equal contiguous runs, so every SM and every warp streams the
+// same number of bytes whatever N and K are.  A row that lies in one run is finished by its warp; the parts of a row
+// that runs share are added in warp order after a barrier: no atomics, bit-identical from run to run.  Each warp keeps
+// 8 - 16 items in flight in registers and requests the first ones before the dependency wait.
+constexpr int kMvWarps = 16, kMvThreads = kMvWarps * 32, kMvBatch = 8;
+
+struct MatvecParams {
+  const uint4* w;
+  const float *bias, *x, *delta, *delta_w, *norm_w;
+  float *y, *x_out;
+  float eps;
+  int N, K, ldw8;        // ldw8: row stride in 16-byte units
+  short act, norm;
+};
+
+__device__ __forceinline__ uint4 ld_stream(const uint4* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+
+__global__ void __launch_bounds__(kMvThreads, 1) matvec_kernel(const MatvecParams p) {
+  extern __shared__ __align__(16) float mv_smem[];
+  __shared__ float red[4 * kMvWarps], part_v[2 * kMvWarps];
+  __shared__ int part_r[2 * kMvWarps];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int KC = (p.K + 255) >> 8;
+  const int unit = p.act == NB_ACT_SWIGLU_PAIRS ? 2 : 1;
+  const int NU = p.N / unit;
+  const int r0 = (int)((long long)NU * blockIdx.x / gridDim.x) * unit, r1 = (int)((long long)NU * (blockIdx.x + 1) / gridDim.x) * unit;
+  const int R = r1 - r0, items = R * KC;
+  const int i0 = (int)((long long)items * warp / kMvWarps), i1 = (int)((long long)items * (warp + 1) / kMvWarps);
+  float* xs = mv_smem;                                  // per 256 columns: first halves of the lanes' eight values, then second halves
+  float* ysum = xs + KC * 256;
+
+  int lr = i0 / KC, lc = i0 - lr * KC, li = i0;         // next item to request
+  const uint4* wp = p.w + (size_t)(r0 + lr) * p.ldw8;   // its row
+  auto request = [&]() -> uint4 {
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (li < i1) {
+      const int c8 = lc * 32 + lane;
+      if (c8 < p.ldw8) v = ld_stream(wp + c8);
+      ++li;
+      if (++lc == KC) { lc = 0; wp += p.ldw8; }
+    }
+    return v;
+  };
+  uint4 cur[kMvBatch];
+#pragma unroll
+  for (int u = 0; u < kMvBatch; ++u) cur[u] = request();
+  for (int r = tid; r < R; r += kMvThreads) ysum[r] = 0.f;
+  if (tid < 2 * kMvWarps) part_r[tid] = -1;
+
+  pdl_enter();
+
+  auto slot = [](int k) { return (k & ~255) + ((k & 4) << 5) + ((k & 255) >> 3) * 4 + (k & 3); };
+  auto each = [&](auto f) {
+    for (int k = tid; k < p.K; k += kMvThreads) f(xs[slot(k)]);
+  };
+  for (int k = p.K + tid; k < KC * 256; k += kMvThreads) xs[slot(k)] = 0.f;
+  float mean, inv;
+  if (p.delta) {
+    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.delta[k];
+    norm_stats<kMvWarps>(p.norm, p.K, p.eps, red, each, mean, inv);
+    for (int k = tid; k < p.K; k += kMvThreads) {
+      const float v = p.x[k] + (xs[slot(k)] - mean) * inv * p.delta_w[k];
+      if (blockIdx.x == 0) p.x_out[k] = v;
+      xs[slot(k)] = v;
+    }
+  } else {
+    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.x[k];
+  }
+  if (p.norm_w) {
+    norm_stats<kMvWarps>(p.norm, p.K, p.eps, red + 2 * kMvWarps, each, mean, inv);
+    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = (xs[slot(k)] - mean) * inv * p.norm_w[k];
+  }
+  __syncthreads();
+
+  int ur = i0 / KC, uc = i0 - ur * KC;                  // next item to multiply
+  int recs = 0;
+  bool whole = uc == 0;                                 // the current row began in this run
+  float acc = 0.f;
+  for (int i = i0; i < i1; i += kMvBatch) {
+    uint4 nxt[kMvBatch];
+#pragma unroll
+    for (int u = 0; u < kMvBatch; ++u) nxt[u] = request();
+#pragma unroll
+    for (int u = 0; u < kMvBatch; ++u) {
+      if (i + u < i1) {
+        const float4 a = *reinterpret_cast<const float4*>(xs + uc * 256 + lane * 4);
+        const float4 b = *reinterpret_cast<const float4*>(xs + uc * 256 + 128 + lane * 4);
+        const uint4 t = cur[u];
+        acc = fmaf(bf_lo(t.x), a.x, acc); acc = fmaf(bf_hi(t.x), a.y, acc);
+        acc = fmaf(bf_lo(t.y), a.z, acc); acc = fmaf(bf_hi(t.y), a.w, acc);
+        acc = fmaf(bf_lo(t.z), b.x, acc); acc = fmaf(bf_hi(t.z), b.y, acc);
+        acc = fmaf(bf_lo(t.w), b.z, acc); acc = fmaf(bf_hi(t.w), b.w, acc);
+        const bool end_row = ++uc == KC;
+        if (end_row || i + u + 1 == i1) {
+          const float s = warp_sum(acc);
+          if (lane == 0) {
+            if (end_row && whole) {
+              ysum[ur] = s;
+            } else {                                    // at most the first and the last row of a run
+              part_v[2 * warp + recs] = s;
+              part_r[2 * warp + recs] = ur;
+            }
+          }
+          if (!(end_row && whole)) ++recs;
+          acc = 0.f;
+          whole = true;
+          if (end_row) { uc = 0; ++ur; }
+        }
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < kMvBatch; ++u) cur[u] = nxt[u];
+  }
+  __syncthreads();
+  auto row_value = [&](int r) {
+    float v = ysum[r];
+#pragma unroll
+    for (int j = 0; j < 2 * kMvWarps; ++j)
+      if (part_r[j] == r) v += part_v[j];
+    return v + (p.bias ? p.bias[r0 + r] : 0.f);
+  };
+  if (unit == 2) {
+    for (int c = tid; c < R / 2; c += kMvThreads) p.y[(r0 >> 1) + c] = silu_f(row_value(2 * c)) * row_value(2 * c + 1);
+  } else {
+    for (int r = tid; r < R; r += kMvThreads) p.y[r0 + r] = row_value(r);
+  }
+}
+
+}  // namespace nb
+
+using namespace nb;
+
+extern "C" int nb_embed_scaled(const void* table_bf16, const int64_t* token, int rows, int V, int C, float scale, float* x, void* stream) {
+  if (!table_bf16 || !token || !x || rows < 1 || V < 1 || C < 1) return NB_ERR_ARG;
+  if (int rc = check_device()) return rc;
+  return launch_pdl(embed_scaled_kernel, dim3(rows), dim3(256), 0, (cudaStream_t)stream, reinterpret_cast<const bf16*>(table_bf16),
+                    reinterpret_cast<const long long*>(token), x, V, C, scale);
+}
+
+extern "C" int nb_residual_norm(float* x, const float* y, const float* wy, const float* w, int norm, float eps, void* h, int h_dtype,
+                                int ldh, int rows, int C, void* stream) {
+  if (!x || (y && !wy) || (h && !w) || (!y && !h) || rows < 1 || C < 1 || (h && ldh < C)) return NB_ERR_ARG;
+  if ((norm != NB_NORM_RMS && norm != NB_NORM_LAYER) || (h_dtype != NB_BF16 && h_dtype != NB_F32)) return NB_ERR_ARG;
+  if (C > 12 * 1024) return NB_ERR_SHAPE;   // the row sits in shared memory
+  if (int rc = check_device()) return rc;
+  const size_t smem = (size_t)C * 4;
+  if (h_dtype == NB_BF16)
+    return launch_pdl(residual_norm_kernel<bf16>, dim3(rows), dim3(kChainThreads), smem, (cudaStream_t)stream, x, y, wy, w, norm, eps,
+                      reinterpret_cast<bf16*>(h), ldh, C);
+  return launch_pdl(residual_norm_kernel<float>, dim3(rows), dim3(kChainThreads), smem, (cudaStream_t)stream, x, y, wy, w, norm, eps,
+                    reinterpret_cast<float*>(h), ldh, C);
+}
+
+extern "C" int nb_linear_f32(const float* x, int ldx, const void* w, int ldw, const float* bias, int act, int M, int N, int K, float* y,
+                             int ldy, void* stream) {
+  if (!x || !w || !y || M < 1 || N < 1 || K < 1 || ldx < K || ldw < K) return NB_ERR_ARG;
+  if (act != NB_ACT_NONE && act != NB_ACT_SWIGLU_PAIRS) return NB_ERR_ARG;
+  if (act == NB_ACT_SWIGLU_PAIRS && N % 2) return NB_ERR_SHAPE;
+  if (ldy < (act == NB_ACT_SWIGLU_PAIRS ? N / 2 : N)) return NB_ERR_ARG;
+  if ((M + kFT - 1) / kFT > 65535) return NB_ERR_SHAPE;
+  if (int rc = check_device()) return rc;
+  linear_f32_kernel<<<dim3((N + kFT - 1) / kFT, (M + kFT - 1) / kFT), 256, 0, (cudaStream_t)stream>>>(
+      x, ldx, reinterpret_cast<const bf16*>(w), ldw, bias, act, M, N, K, y, ldy);
+  return check_launch();
+}
+
+extern "C" int nb_matvec_bf16(const nb_matvec_args* a, void* stream) {
+  if (!a || !a->w || !a->x || !a->y || a->N < 1 || a->K < 1 || a->ldw < a->K) return NB_ERR_ARG;
+  if (a->delta && (!a->delta_w || !a->x_out || !a->norm_w || a->x_out == a->x)) return NB_ERR_ARG;
+  if (a->norm != NB_NORM_RMS && a->norm != NB_NORM_LAYER) return NB_ERR_ARG;
+  if (a->act != NB_ACT_NONE && a->act != NB_ACT_SWIGLU_PAIRS) return NB_ERR_ARG;
+  const int unit = a->act == NB_ACT_SWIGLU_PAIRS ? 2 : 1;
+  if (a->N % unit) return NB_ERR_SHAPE;
+  if ((uintptr_t)a->w % 16 || a->ldw % 8) return NB_ERR_ALIGN;
+  if (int rc = check_device()) return rc;
+  const int G = std::min(sm_count(), a->N / unit);
+  const int rows = ((a->N / unit + G - 1) / G) * unit, kc = (a->K + 255) / 256;
+  const size_t smem = ((size_t)kc * 256 + rows) * 4;
+  constexpr size_t kMax = 200 * 1024;
+  if (smem > kMax) return NB_ERR_SHAPE;
+  static bool attr_done[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!attr_done[dev & 63]) {
+    if (cudaError_t e = cudaFuncSetAttribute(matvec_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMax)) return record_cuda_error(e);
+    attr_done[dev & 63] = true;
+  }
+  MatvecParams p;
+  p.w = reinterpret_cast<const uint4*>(a->w);
+  p.bias = a->bias; p.x = a->x; p.delta = a->delta; p.delta_w = a->delta_w; p.norm_w = a->norm_w;
+  p.y = a->y; p.x_out = a->x_out;
+  p.eps = a->eps; p.N = a->N; p.K = a->K; p.ldw8 = a->ldw / 8;
+  p.act = (short)a->act; p.norm = (short)a->norm;
+  return launch_pdl(matvec_kernel, dim3(G), dim3(kMvThreads), smem, (cudaStream_t)stream, p);
+}

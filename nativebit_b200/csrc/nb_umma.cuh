@@ -90,12 +90,13 @@ inline EncodeTiledFn encode_fn() {
   return fn;
 }
 
-// (rows, cols) row-major bf16 matrix -> tensor map with a (box_rows x 64) box and 128-byte swizzle.
-inline int make_map(CUtensorMap* map, const void* base, int rows, int cols, int box_rows) {
+// (rows, cols) row-major bf16 matrix, rows `ld` elements apart (0: cols; a multiple of 8) -> tensor map with a
+// (box_rows x 64) box and 128-byte swizzle.  Boxes past the last row or column are filled with zeros.
+inline int make_map(CUtensorMap* map, const void* base, int rows, int cols, int box_rows, int ld = 0) {
   EncodeTiledFn fn = encode_fn();
   if (!fn) { set_last_error("cuTensorMapEncodeTiled is not available from the driver"); return NB_ERR_LAUNCH; }
   const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
-  const cuuint64_t strides[1] = {(cuuint64_t)cols * 2};
+  const cuuint64_t strides[1] = {(cuuint64_t)(ld ? ld : cols) * 2};
   const cuuint32_t box[2] = {(cuuint32_t)kBK, (cuuint32_t)box_rows};
   const cuuint32_t estr[2] = {1, 1};
   const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,

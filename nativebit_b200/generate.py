@@ -26,6 +26,7 @@ import torch.nn.functional as F
 
 from . import ops, synthetic, tp
 from .packed_linear import PackedLinear
+from .session import Session
 
 
 @dataclass
@@ -257,6 +258,9 @@ class PackedGPT(torch.nn.Module):
         return (logits, new_caches) if kv_caches is not None else logits
 
     # ------------------------------------------------------------------ construction
+    def session(self, batch_size: int = 1, **options) -> "DecodeSession":
+        return DecodeSession(self, batch_size, **options)
+
     @staticmethod
     def random_init(config: ModelConfig, seed: int = 0, device="cuda", tp_rank: int = 0, tp_size: int = 1, group=None):
         """Seeded random-init model: every rank generates the same global packed weights (per-layer
@@ -325,8 +329,8 @@ def step(model: PackedGPT, x: torch.Tensor, caches):
     return logits[:, -1, :], caches
 
 
-class DecodeSession:
-    """Greedy decoding with the whole step in one CUDA graph: token, position and caches live on the
+class DecodeSession(Session):
+    """Greedy decoding of a PackedGPT with the whole step in one CUDA graph: token, position and caches live on the
     device, the next token is the argmax written back into the token buffer, so N steps are N graph
     replays without a host round trip.  Attention in the captured step covers the full context
     buffer under a position mask (static shapes), as the reference's cached path does
@@ -334,7 +338,7 @@ class DecodeSession:
 
     def __init__(self, model: PackedGPT, batch_size: int = 1, use_graph: bool = True, fused: bool = True,
                  batch_gemm: bool = False, stream: bool | None = None, tile_gemv: bool | None = None, hand_head: bool = True):
-        self.model, self.B = model, batch_size
+        super().__init__(model, batch_size, model.context_len, model.config.vocab_size, model.embedding.device, use_graph)
         self.hand_head = hand_head            # False: the LM head of a single sequence stays a library GEMM (comparison)
         self.residual_in_matvec = False       # True: out_proj and down add into the residual stream themselves (flag 4 of
                                               # nb_gemv_stream) instead of the next norm prologue: bit-identical, measured neutral
@@ -363,18 +367,9 @@ class DecodeSession:
                 raise RuntimeError("the one-launch decode step needs batch 1, one rank, bf16 embeddings and block-128 codebooks")
         self.prog = None
         self.batch_gemm = batch_gemm          # kept for compatibility: batches above 16 rows always take the tensor-core kernel
-        dev = model.embedding.device
-        self.dev = dev
+        dev = self.dev
         self.caches = init_kv_cache(model, batch_size, dev)
-        self.pos = torch.zeros(1, dtype=torch.long, device=dev)
-        self.pos_host = 0                     # the same position, tracked on the host: steps past the context are refused
-        self.token = torch.zeros(batch_size, 1, dtype=torch.long, device=dev)
-        self.logits = torch.zeros(batch_size, model.config.vocab_size, dtype=torch.float32, device=dev)
         self.k_idx = torch.arange(model.context_len, device=dev)
-        self.use_graph = use_graph
-        self.graph = None
-        self._prefill_graphs = {}             # prompt length -> (captured prefill, its static input)
-        self.stream = torch.cuda.Stream(device=dev)
         if fused:  # static activation buffers of the fused step
             cfg, B = model.config, batch_size
             f32 = dict(dtype=torch.float32, device=dev)
@@ -504,44 +499,18 @@ class DecodeSession:
             logits = m._head(self.bh)                            # the LM head is a plain library GEMM (bf16 table, 164 MB)
         ops.softcap_argmax(logits, cfg.logit_cap, self.logits, self.token, self.pos)
 
-    @torch.no_grad()
-    def prefill(self, prompt: torch.Tensor) -> torch.Tensor:
-        """prompt (B, T): fills the caches, sets the position and the first generated token."""
-        if prompt.shape[1] > self.model.context_len:
-            raise RuntimeError(f"prompt of {prompt.shape[1]} tokens exceeds the context of {self.model.context_len}")
-        T = int(prompt.shape[1])
-        if not self.use_graph or not prompt.is_cuda:
-            self._prefill_body(prompt)
-        else:
-            # one CUDA graph per prompt length: the eager forward is about thirty small launches per layer and
-            # is bound by the host; replayed from a graph only the device time remains
-            entry = self._prefill_graphs.get(T)
-            cur = torch.cuda.current_stream(self.dev)
-            if entry is None:
-                static_in = prompt.clone()
-                self.stream.wait_stream(cur)
-                with torch.cuda.stream(self.stream):
-                    self._prefill_body(static_in)            # warms every kernel up and IS this call's result
-                    self.stream.synchronize()
-                    g = torch.cuda.CUDAGraph()
-                    with torch.cuda.graph(g, stream=self.stream):
-                        self._prefill_body(static_in)
-                cur.wait_stream(self.stream)
-                self._prefill_graphs[T] = (g, static_in)
-            else:
-                g, static_in = entry
-                static_in.copy_(prompt)
-                g.replay()
-        self.caches = [(k, v, T) for k, v, _ in self.caches]
-        self.pos_host = T
-        return self.logits
-
     def _prefill_body(self, prompt: torch.Tensor) -> None:
         caches = [(k, v, 0) for k, v, _ in self.caches]
         logits, _ = self.model(prompt, kv_caches=caches, last_only=True)      # the caches are written in place
         self.pos.fill_(prompt.shape[1])
         self.logits.copy_(logits[:, -1, :])
         self.token.copy_(self.logits.argmax(-1, keepdim=True))
+
+    def _extend_body(self, tokens: torch.Tensor, want: list[int]) -> torch.Tensor:
+        logits, _ = self.model(tokens, kv_caches=[(k, v, self.pos_host) for k, v, _ in self.caches])
+        self.logits.copy_(logits[:, -1, :])
+        self.token.copy_(self.logits.argmax(-1, keepdim=True))
+        return logits[:, want, :]
 
     @torch.no_grad()
     def _step_body(self):
@@ -581,44 +550,6 @@ class DecodeSession:
             obj = getattr(self.model, name, None)
             if obj is not None and int(obj.status.item()) != 0:
                 raise RuntimeError(f"{name}: a peer did not arrive within the bounded wait")
-
-    def step(self) -> None:
-        """One decode step for every sequence: consumes self.token, leaves the next token there.
-        Raises (before anything is launched) when the cache has no free slot left."""
-        ctx = self.model.context_len
-        if self.pos_host >= ctx:
-            raise RuntimeError(f"decode position {self.pos_host} is past the end of the context ({ctx}): the KV cache is full")
-        if not self.use_graph:
-            self._step_body()
-            self.pos_host += 1
-            return
-        if self.graph is None:
-            # the warm-up and the capture run on the session's stream: it must first see what the caller's
-            # stream has written (prefill: caches, position, first token)
-            self.stream.wait_stream(torch.cuda.current_stream())
-            with torch.cuda.stream(self.stream):
-                saved = (self.pos.clone(), self.token.clone(), self.logits.clone())
-                for _ in range(min(2, ctx - self.pos_host)):      # warm-up outside capture, inside the context
-                    self._step_body()
-                self.stream.synchronize()
-                self.pos.copy_(saved[0]); self.token.copy_(saved[1]); self.logits.copy_(saved[2])
-                self.graph = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(self.graph, stream=self.stream):
-                    self._step_body()
-                # the capture does not execute: state is unchanged; stale cache slots past `pos` are masked
-            torch.cuda.current_stream().wait_stream(self.stream)
-        self.graph.replay()
-        self.pos_host += 1
-
-    @torch.no_grad()
-    def generate(self, prompt: torch.Tensor, n_generate: int) -> torch.Tensor:
-        """Greedy continuation (B, n_generate) of prompt (B, T)."""
-        self.prefill(prompt)
-        out = [self.token.clone()]
-        for _ in range(n_generate - 1):
-            self.step()
-            out.append(self.token.clone())
-        return torch.cat(out, dim=1)
 
 
 def benchmark(model: PackedGPT, prompt_tokens, n_generate: int = 128, n_runs: int = 3, device="cuda", batch_size: int = 1,
@@ -700,3 +631,12 @@ def load_packed_model(packed_path: str, config, device="cuda", tp_rank: int = 0,
     lnf = params.get("params/ln_f/weight")
     lnf_t = torch.from_numpy(lnf.astype(np.float32)).to(dev) if lnf is not None else torch.ones(C, device=dev)
     return PackedGPT(cfg, emb_t, blocks, lnf_t, tp_rank, tp_size, group)
+
+
+def load_folder(folder: str, config: dict, dtype: torch.dtype, context_len: int, device) -> PackedGPT:
+    """A model folder's packed decoder: config.json with ModelConfig's fields, weights in model.nbpack.npz.  The context
+    is the smaller of the configuration's and the one asked for."""
+    fields = {k: config[k] for k in ModelConfig.__dataclass_fields__ if k in config}
+    cfg = ModelConfig(**fields)
+    cfg.context_len = min(cfg.context_len, context_len)
+    return load_packed_model(f"{folder}/model.nbpack.npz", cfg, device)
