@@ -58,7 +58,7 @@ int nb_matvec_bf16(const nb_matvec_args* a, void* stream);
 
 /* ---- latent attention -------------------------------------------------------------------------------------
  * Cache of a layer: (B, ctx, ldc) rows [latent (rank) | rotated key part (rot)] of the activation dtype, ldc a
- * multiple of 8.  cos2 / sin2: (ctx, rot) fp32, every pair's entry twice (interleaved pairs).
+ * multiple of 8, columns past them zero.  cos2 / sin2: (ctx, rot) fp32, every pair's entry twice (interleaved pairs).
  *
  * nb_latent_prepare, per row b * T + t: cq = RMSNorm(a[q_off ..]) * q_norm (q_rank values); if kv_off >= 0:
  * cache[b][pos0 + t] = [RMSNorm(a[kv_off ..]) * kv_norm | rotate(a[kv_off + rank ..])]. */

@@ -13,6 +13,7 @@
 #include <algorithm>
 
 #include "nb_layered.cuh"
+#include "nb_mma.cuh"
 
 namespace nb {
 
@@ -117,13 +118,25 @@ __global__ void __launch_bounds__(256) gla_scan_kernel(const nb_gla_args p, GlaW
   const int b = bh / p.H, h = bh - b * p.H, d = i / (p.lds / 4);
   float4* st = reinterpret_cast<float4*>(p.state) + (size_t)bh * per + i;
   float4 s = *st;
-  for (int n = 0; n < chunks; ++n) {
-    const size_t head = ((size_t)b * chunks + n) * p.H + h;
-    float4* up = reinterpret_cast<float4*>(w.u) + head * per + i;
-    const float a = expf(w.dec[head * p.dim + d]);
-    const float4 u = *up;
-    *up = s;
-    s.x = fmaf(s.x, a, u.x); s.y = fmaf(s.y, a, u.y); s.z = fmaf(s.z, a, u.z); s.w = fmaf(s.w, a, u.w);
+  constexpr int kAhead = 8;            // chunks requested at a time: the loads do not depend on one another
+  for (int n0 = 0; n0 < chunks; n0 += kAhead) {
+    float4 u[kAhead];
+    float a[kAhead];
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      const size_t head = ((size_t)b * chunks + min(n0 + j, chunks - 1)) * p.H + h;
+      u[j] = reinterpret_cast<const float4*>(w.u)[head * per + i];
+      a[j] = w.dec[head * p.dim + d];
+    }
+#pragma unroll
+    for (int j = 0; j < kAhead; ++j) {
+      if (n0 + j < chunks) {
+        const size_t head = ((size_t)b * chunks + n0 + j) * p.H + h;
+        reinterpret_cast<float4*>(w.u)[head * per + i] = s;
+        const float e = expf(a[j]);
+        s.x = fmaf(s.x, e, u[j].x); s.y = fmaf(s.y, e, u[j].y); s.z = fmaf(s.z, e, u[j].z); s.w = fmaf(s.w, e, u[j].w);
+      }
+    }
   }
   *st = s;
 }
@@ -275,9 +288,340 @@ template <typename T> __global__ void __launch_bounds__(256) gla_finish_kernel(c
   for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * inv * p.norm_w[i] * silu_f(to_f(g[i])));
 }
 
+// ---- the same two kernels for bf16 projections on the tensor cores.  q, k and v are bf16 as they are; everything the
+// recurrence adds — decayed q and k, the state, the scores — stays fp32 and enters a product as two bf16 terms (the
+// product of two such pairs as three).  Four warps per CTA; vdim <= VD.
+constexpr int kGmThreads = 128;
+constexpr int kGmLd = 64 + 8;          // row stride of a staged tile of 64 channels, in elements
+constexpr float kSplitLimit = -60.f;   // a sub-block that decays further is taken pair by pair
+
+template <int VD> struct GlaStateSmem {
+  bf16 khi[kGC * kGmLd], klo[kGC * kGmLd], v[kGC * (VD + 8)];
+  float tot[kGSubs * 64];
+};
+
+// Copies rows of `cols` bf16 (zero past `valid` columns and `cnt` rows) into shared memory; vec: 16-byte aligned, cols % 8 == 0.
+__device__ __forceinline__ void stage_rows(bf16* dst, int ldd, const bf16* src, int lds, int cols, int valid, int cnt, bool vec) {
+  if (vec) {
+    const int c8 = (threadIdx.x & 7) * 8;
+    for (int t = threadIdx.x >> 3; t < kGC; t += kGmThreads / 8)
+      for (int c = c8; c < cols; c += 64) {
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (t < cnt && c < valid) v = *reinterpret_cast<const uint4*>(src + (size_t)t * lds + c);
+        *reinterpret_cast<uint4*>(dst + t * ldd + c) = v;
+      }
+  } else {
+    for (int i = threadIdx.x; i < kGC * cols; i += kGmThreads) {
+      const int t = i / cols, c = i - t * cols;
+      dst[t * ldd + c] = (t < cnt && c < valid) ? src[(size_t)t * lds + c] : from_f<bf16>(0.f);
+    }
+  }
+}
+
+// grid (chunks, H * d tiles, B): 64 channels x vdim of a chunk's contribution.
+template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_kernel(const nb_gla_args p, GlaWs w, int dtiles, int vec) {
+  extern __shared__ __align__(16) uint8_t gsm_raw[];
+  GlaStateSmem<VD>& sm = *reinterpret_cast<GlaStateSmem<VD>*>(gsm_raw);
+  const int n = blockIdx.x, h = blockIdx.y / dtiles, d0 = (blockIdx.y - h * dtiles) * 64, b = blockIdx.z;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t0 = n * kGC, cnt = min(kGC, p.T - t0), HD = p.H * p.dim;
+  const bf16* base = reinterpret_cast<const bf16*>(p.p) + (size_t)(b * p.T + t0) * p.ldp;
+  const float* bl = w.bl + (size_t)(b * p.T + t0) * HD + h * p.dim + d0;
+  const int dn = min(64, p.dim - d0);
+  for (int i = tid; i < kGSubs * 64; i += kGmThreads) {
+    const int s = i >> 6, d = i & 63, t = min(cnt, (s + 1) * kGS) - 1;
+    sm.tot[i] = (s * kGS < cnt && d < dn) ? bl[(size_t)t * HD + d] : 0.f;
+  }
+  stage_rows(sm.v, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  __syncthreads();
+  const bf16* kp = base + p.k_off + h * p.dim + d0;
+#pragma unroll 4
+  for (int i = tid; i < kGC * 32; i += kGmThreads) {      // pairs of channels
+    const int t = i >> 5, d = (i & 31) * 2, s = t / kGS;
+    float x = 0.f, y = 0.f;
+    if (t < cnt) {
+      if (d < dn) {
+        float e = sm.tot[s * 64 + d] - bl[(size_t)t * HD + d];
+        for (int m = s + 1; m < kGSubs; ++m) e += sm.tot[m * 64 + d];
+        x = to_f(kp[(size_t)t * p.ldp + d]) * expf(e);
+      }
+      if (d + 1 < dn) {
+        float e = sm.tot[s * 64 + d + 1] - bl[(size_t)t * HD + d + 1];
+        for (int m = s + 1; m < kGSubs; ++m) e += sm.tot[m * 64 + d + 1];
+        y = to_f(kp[(size_t)t * p.ldp + d + 1]) * expf(e);
+      }
+    }
+    uint32_t hi, lo;
+    split_bf16(x, y, hi, lo);
+    *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
+    *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
+  }
+  __syncthreads();
+  float acc[VD / 8][4];
+#pragma unroll
+  for (int i = 0; i < VD / 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  // rows of the product are channels: the A fragment is k transposed
+  const int at = ((lane >> 4) << 3) + (lane & 7), ac = warp * 16 + ((lane >> 3) & 1) * 8;
+#pragma unroll
+  for (int kk = 0; kk < kGC; kk += 16) {
+    uint32_t hi[4], lo[4];
+    ldsm_x4_t(hi, sm.khi + (kk + at) * kGmLd + ac);
+    ldsm_x4_t(lo, sm.klo + (kk + at) * kGmLd + ac);
+#pragma unroll
+    for (int v = 0; v < VD / 16; ++v) {
+      uint32_t bb[4];
+      ldsm_x4_t(bb, sm.v + (kk + (lane & 15)) * (VD + 8) + v * 16 + (lane >> 4) * 8);
+      mma_bf16(acc[2 * v], hi, bb[0], bb[1]);
+      mma_bf16(acc[2 * v + 1], hi, bb[2], bb[3]);
+      mma_bf16(acc[2 * v], lo, bb[0], bb[1]);
+      mma_bf16(acc[2 * v + 1], lo, bb[2], bb[3]);
+    }
+  }
+  const size_t head = ((size_t)b * gridDim.x + n) * p.H + h;
+  float* u = w.u + (head * p.dim + d0) * p.lds;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int d = warp * 16 + (lane >> 2) + 8 * half;
+    if (d < dn) {
+#pragma unroll
+      for (int i = 0; i < VD / 8; ++i) {
+        const int v = i * 8 + (lane & 3) * 2;              // lds is a multiple of 4: a pair never straddles the end
+        if (v < p.lds) *reinterpret_cast<float2*>(u + (size_t)d * p.lds + v) = make_float2(acc[i][2 * half], acc[i][2 * half + 1]);
+      }
+    }
+  }
+  if (tid < dn) w.dec[head * p.dim + d0 + tid] = sm.tot[tid] + sm.tot[64 + tid] + sm.tot[128 + tid] + sm.tot[192 + tid];
+}
+
+template <int VD> struct GlaOutSmem {
+  bf16 q[kGC * kGmLd], k[kGC * kGmLd];           // as they are
+  bf16 khi[kGC * kGmLd], klo[kGC * kGmLd];       // k decayed to the end of its sub-block
+  float bl[kGC * 68];                            // summed log decays
+  float tot[kGSubs * 64];                        // log decay of a whole sub-block
+  float fac[10 * 64];                            // factors of the block pairs and of the chunk's start, see below
+  bf16 shi[64 * (VD + 8)], slo[64 * (VD + 8)];   // a tile of the state; at the end v
+};
+
+// grid (chunks, H, B).  Warp i owns sub-block i: its 16 queries against the keys of sub-blocks 0 .. i and against the state
+// at the chunk's start; then the scores against the values, the norm over the head's outputs and the gate.
+//   q . k over sub-blocks i > j: (q exp(bl)) . (k exp(tot_j - bl)) * exp(tot_{j+1} + .. + tot_{i-1}), the last on q's side;
+//   i == j: the same with exp(-tot_i), as long as no channel of the tile decays past kSplitLimit inside the sub-block.
+template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_kernel(const nb_gla_args p, GlaWs w, int vec) {
+  extern __shared__ __align__(16) uint8_t gsm_raw[];
+  GlaOutSmem<VD>& sm = *reinterpret_cast<GlaOutSmem<VD>*>(gsm_raw);
+  const int n = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int t0 = n * kGC, cnt = min(kGC, p.T - t0), HD = p.H * p.dim;
+  const bf16* base = reinterpret_cast<const bf16*>(p.p) + (size_t)(b * p.T + t0) * p.ldp;
+  const float* blg = w.bl + (size_t)(b * p.T + t0) * HD + h * p.dim;
+  const float* S = w.u + (((size_t)b * gridDim.x + n) * p.H + h) * p.dim * p.lds;
+  const float qscale = 1.0f / sqrtf((float)p.dim);
+  const int ra = warp * 16 + (lane >> 2), rb = ra + 8, c2 = (lane & 3) * 2;   // this lane's two query rows, its column pair
+
+  float sc[kGSubs][2][4];              // scores: key sub-block, half of it, fragment
+  float o[VD / 8][4];
+#pragma unroll
+  for (int j = 0; j < kGSubs; ++j)
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[j][x][e] = 0.f;
+#pragma unroll
+  for (int i = 0; i < VD / 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[i][e] = 0.f;
+
+  for (int d0 = 0; d0 < p.dim; d0 += 64) {
+    const int dn = min(64, p.dim - d0);
+    __syncthreads();                   // the tile before is no longer read
+    stage_rows(sm.q, kGmLd, base + p.q_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
+    stage_rows(sm.k, kGmLd, base + p.k_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
+    for (int i = tid; i < kGC * 64; i += kGmThreads) {
+      const int t = i >> 6, d = i & 63;
+      sm.bl[t * 68 + d] = (t < cnt && d < dn) ? blg[(size_t)t * HD + d0 + d] : 0.f;
+    }
+    for (int i = tid; i < 64 * (VD / 2); i += kGmThreads) {     // state, in pairs of columns
+      const int d = i / (VD / 2), v = (i - d * (VD / 2)) * 2;
+      float2 x = make_float2(0.f, 0.f);
+      if (d < dn && v < p.lds) x = *reinterpret_cast<const float2*>(S + (size_t)(d0 + d) * p.lds + v);
+      uint32_t hi, lo;
+      split_bf16(x.x, x.y, hi, lo);
+      *reinterpret_cast<uint32_t*>(sm.shi + d * (VD + 8) + v) = hi;
+      *reinterpret_cast<uint32_t*>(sm.slo + d * (VD + 8) + v) = lo;
+    }
+    __syncthreads();
+    bool deep = false;                 // some channel of the tile decays past the limit inside a sub-block
+    for (int i = tid; i < kGSubs * 64; i += kGmThreads) {
+      const int s = i >> 6, t = min(cnt, (s + 1) * kGS) - 1;
+      const float x = s * kGS < cnt ? sm.bl[t * 68 + (i & 63)] : 0.f;
+      sm.tot[i] = x;
+      deep |= x < kSplitLimit;
+    }
+    deep = __syncthreads_or(deep);
+    if (tid < 64) {
+      const float a0 = sm.tot[tid], a1 = sm.tot[64 + tid], a2 = sm.tot[128 + tid], a3 = sm.tot[192 + tid];
+      float* f = sm.fac + tid;
+      f[0 * 64] = expf(a1);            // between sub-blocks 2 and 0
+      f[1 * 64] = expf(a2);            // 3 and 1
+      f[2 * 64] = expf(a1 + a2);       // 3 and 0
+      f[3 * 64] = expf(a0);            // from the chunk's start to sub-block 1, 2, 3
+      f[4 * 64] = expf(a0 + a1);
+      f[5 * 64] = expf(a0 + a1 + a2);
+      f[6 * 64] = deep ? 0.f : expf(-a0);      // inside sub-block 0 .. 3
+      f[7 * 64] = deep ? 0.f : expf(-a1);
+      f[8 * 64] = deep ? 0.f : expf(-a2);
+      f[9 * 64] = deep ? 0.f : expf(-a3);
+    }
+    for (int i = tid; i < kGC * 32; i += kGmThreads) {
+      const int t = i >> 5, d = (i & 31) * 2;
+      const uint32_t kk = *reinterpret_cast<const uint32_t*>(sm.k + t * kGmLd + d);
+      const float* tt = sm.tot + (t / kGS) * 64 + d;
+      uint32_t hi, lo;
+      split_bf16(bf_lo(kk) * expf(tt[0] - sm.bl[t * 68 + d]), bf_hi(kk) * expf(tt[1] - sm.bl[t * 68 + d + 1]), hi, lo);
+      if (t >= cnt) hi = lo = 0u;
+      *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
+      *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int kk = 0; kk < 64; kk += 16) {
+      if (kk >= dn) break;
+      // decayed queries of this step, fp32, in the A fragment's places: (row a, row b) x (columns c2, c2 + 8)
+      float qd[4][2];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int r = (j & 1) ? rb : ra, c = kk + c2 + (j >> 1) * 8;
+        const uint32_t qq = *reinterpret_cast<const uint32_t*>(sm.q + r * kGmLd + c);
+        qd[j][0] = bf_lo(qq) * qscale * expf(sm.bl[r * 68 + c]);
+        qd[j][1] = bf_hi(qq) * qscale * expf(sm.bl[r * 68 + c + 1]);
+      }
+      auto fragment = [&](const float* f, uint32_t (&hi)[4], uint32_t (&lo)[4]) {   // f: per-channel factor or null
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int c = kk + c2 + (j >> 1) * 8;
+          const float fx = f ? f[c] : 1.f, fy = f ? f[c + 1] : 1.f;
+          split_bf16(qd[j][0] * fx, qd[j][1] * fy, hi[j], lo[j]);
+        }
+      };
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int j = 0; j < kGSubs; ++j) {
+        if (j > warp) break;
+        const float* f = j == warp ? sm.fac + (6 + warp) * 64
+                         : j + 1 == warp ? nullptr
+                         : sm.fac + (warp == 2 ? 0 : j == 1 ? 1 : 2) * 64;
+        if (j == warp && deep) continue;
+        fragment(f, hi, lo);
+        uint32_t kh[4], kl[4];         // sixteen keys: row = token, column = channel
+        const int off = (j * 16 + (lane & 7) + ((lane >> 4) << 3)) * kGmLd + kk + ((lane >> 3) & 1) * 8;
+        ldsm_x4(kh, sm.khi + off);
+        ldsm_x4(kl, sm.klo + off);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          mma_bf16(sc[j][x], hi, kh[2 * x], kh[2 * x + 1]);
+          mma_bf16(sc[j][x], hi, kl[2 * x], kl[2 * x + 1]);
+          mma_bf16(sc[j][x], lo, kh[2 * x], kh[2 * x + 1]);
+        }
+      }
+      fragment(warp == 0 ? nullptr : sm.fac + (2 + warp) * 64, hi, lo);
+#pragma unroll
+      for (int v = 0; v < VD / 16; ++v) {
+        uint32_t sh[4], sl[4];
+        const int off = (kk + (lane & 15)) * (VD + 8) + v * 16 + (lane >> 4) * 8;
+        ldsm_x4_t(sh, sm.shi + off);
+        ldsm_x4_t(sl, sm.slo + off);
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          mma_bf16(o[2 * v + x], hi, sh[2 * x], sh[2 * x + 1]);
+          mma_bf16(o[2 * v + x], hi, sl[2 * x], sl[2 * x + 1]);
+          mma_bf16(o[2 * v + x], lo, sh[2 * x], sh[2 * x + 1]);
+        }
+      }
+    }
+    if (deep) {                        // the pairs of this warp's own sub-block, one exponential each
+#pragma unroll
+      for (int j = 0; j < kGSubs; ++j) {
+        if (j != warp) continue;
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int t = e < 2 ? ra : rb, s = j * 16 + x * 8 + c2 + (e & 1);
+            if (s > t || t >= cnt) continue;
+            float sum = 0.f;
+            for (int d = 0; d < dn; ++d)
+              sum += to_f(sm.q[t * kGmLd + d]) * expf(sm.bl[t * 68 + d] - sm.bl[s * 68 + d]) * to_f(sm.k[s * kGmLd + d]);
+            sc[j][x][e] += sum * qscale;
+          }
+      }
+    }
+  }
+  __syncthreads();
+  stage_rows(sm.shi, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < kGSubs; ++j) {
+    if (j > warp) break;
+    uint32_t hi[4], lo[4];
+#pragma unroll
+    for (int f = 0; f < 4; ++f) {
+      const int half = f & 1, x = f >> 1, t = half ? rb : ra, s = j * 16 + x * 8 + c2;
+      const float u = s <= t ? sc[j][x][2 * half] : 0.f, v = s + 1 <= t ? sc[j][x][2 * half + 1] : 0.f;
+      split_bf16(u, v, hi[f], lo[f]);
+    }
+#pragma unroll
+    for (int v = 0; v < VD / 16; ++v) {
+      uint32_t bb[4];
+      ldsm_x4_t(bb, sm.shi + (j * 16 + (lane & 15)) * (VD + 8) + v * 16 + (lane >> 4) * 8);
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        mma_bf16(o[2 * v + x], hi, bb[2 * x], bb[2 * x + 1]);
+        mma_bf16(o[2 * v + x], lo, bb[2 * x], bb[2 * x + 1]);
+      }
+    }
+  }
+  float sa = 0.f, sb = 0.f;            // columns past vdim are zero
+#pragma unroll
+  for (int i = 0; i < VD / 8; ++i) {
+    sa += o[i][0] * o[i][0] + o[i][1] * o[i][1];
+    sb += o[i][2] * o[i][2] + o[i][3] * o[i][3];
+  }
+#pragma unroll
+  for (int x = 1; x < 4; x <<= 1) {
+    sa += __shfl_xor_sync(0xffffffffu, sa, x);
+    sb += __shfl_xor_sync(0xffffffffu, sb, x);
+  }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int t = half ? rb : ra;
+    if (t >= cnt) continue;
+    const float inv = 1.0f / sqrtf((half ? sb : sa) / (float)p.vdim + p.eps);
+    const bf16* g = base + (size_t)t * p.ldp + p.g_off + h * p.vdim;
+    bf16* out = reinterpret_cast<bf16*>(p.out) + (size_t)(b * p.T + t0 + t) * p.ldo + h * p.vdim;
+#pragma unroll
+    for (int i = 0; i < VD / 8; ++i) {
+      const int v = i * 8 + c2;
+      if (vec) {
+        if (v < p.vdim) {
+          const uint32_t gg = *reinterpret_cast<const uint32_t*>(g + v);
+          *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(o[i][2 * half] * inv * p.norm_w[v] * silu_f(bf_lo(gg)),
+                                                            o[i][2 * half + 1] * inv * p.norm_w[v + 1] * silu_f(bf_hi(gg)));
+        }
+      } else {
+        if (v < p.vdim) out[v] = from_f<bf16>(o[i][2 * half] * inv * p.norm_w[v] * silu_f(to_f(g[v])));
+        if (v + 1 < p.vdim) out[v + 1] = from_f<bf16>(o[i][2 * half + 1] * inv * p.norm_w[v + 1] * silu_f(to_f(g[v + 1])));
+      }
+    }
+  }
+}
+
 // ---- one token per sequence.  grid (H, B, S) in clusters of S CTAs along z: a CTA owns a range of value columns of the
 // head's state, reads it once and writes it once; the squares of the outputs are summed over the cluster for the norm.
+// The state was written in the step before (or by the prompt), so it is requested ahead of the dependency wait, and so are
+// the decay's weights, as far as they fit the registers.
 constexpr int kGdThreads = 256, kGdWarps = kGdThreads / 32;
+constexpr int kGdPre = 8;              // rows of the state (four columns each) a thread may hold ahead of the wait
 
 __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_args p) {
   extern __shared__ __align__(16) float gdm[];
@@ -291,37 +635,75 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_arg
   float* qs = ks + p.dim;              // [dim]
   float* os = qs + p.dim;              // [4 * qper] outputs
   float4* part = reinterpret_cast<float4*>(gdm + ((3 * p.dim + 4 * qper + 3) & ~3));   // [kGdThreads]
+  float4* st = reinterpret_cast<float4*>(p.state) + ((size_t)b * p.H + h) * p.dim * quads;
+  const int cols0 = min(cn, kGdThreads), groups0 = cols0 ? kGdThreads / cols0 : 1, g0 = cols0 ? tid / cols0 : 0, cc0 = cols0 ? tid - g0 * cols0 : 0;
+  const bool pre = cn > 0 && cn <= kGdThreads && (p.dim + groups0 - 1) / groups0 <= kGdPre;
+  float4 sreg[kGdPre];
+#pragma unroll
+  for (int i = 0; i < kGdPre; ++i) {
+    const int d = g0 + i * groups0;
+    sreg[i] = (pre && g0 < groups0 && d < p.dim) ? st[(size_t)d * quads + c0 + cc0] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const bool short_rank = p.lda2 <= 16 && p.dim <= kGdThreads;   // a row of W_a2 is one or two 16-byte loads
+  const bf16* w2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)(h * p.dim) * p.lda2;
+  uint4 wa = make_uint4(0u, 0u, 0u, 0u), wb = wa;
+  float bias = 0.f;
+  if (short_rank && tid < p.dim) {
+    wa = *reinterpret_cast<const uint4*>(w2 + (size_t)tid * p.lda2);
+    if (p.lda2 > 8) wb = *reinterpret_cast<const uint4*>(w2 + (size_t)tid * p.lda2 + 8);
+    bias = p.a2_b[h * p.dim + tid];
+  }
   pdl_enter();
   const float* row = reinterpret_cast<const float*>(p.p) + (size_t)b * p.ldp;
+  const float* vrow = row + p.v_off + h * p.vdim;
   const float qscale = 1.0f / sqrtf((float)p.dim);
+  const int vp = 4 * (c0 + cc0);
+  float4 vpre = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (pre && g0 < groups0)
+    vpre = make_float4(vp < p.vdim ? vrow[vp] : 0.f, vp + 1 < p.vdim ? vrow[vp + 1] : 0.f, vp + 2 < p.vdim ? vrow[vp + 2] : 0.f,
+                       vp + 3 < p.vdim ? vrow[vp + 3] : 0.f);
   for (int d = tid; d < p.dim; d += kGdThreads) {
     const int ch = h * p.dim + d;
-    const bf16* w2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)ch * p.lda2;
-    float z = p.a2_b[ch];
-    for (int r = 0; r < p.a_rank; ++r) z = fmaf(to_f(w2[r]), row[p.a_off + r], z);
+    const float k = row[p.k_off + ch], q = row[p.q_off + ch];
+    float z;
+    if (short_rank) {
+      z = bias;
+      const uint32_t u[8] = {wa.x, wa.y, wa.z, wa.w, wb.x, wb.y, wb.z, wb.w};
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        if (2 * r < p.a_rank) z = fmaf(bf_lo(u[r]), row[p.a_off + 2 * r], z);
+        if (2 * r + 1 < p.a_rank) z = fmaf(bf_hi(u[r]), row[p.a_off + 2 * r + 1], z);
+      }
+    } else {
+      z = p.a2_b[ch];
+      for (int r = 0; r < p.a_rank; ++r) z = fmaf(to_f(w2[(size_t)d * p.lda2 + r]), row[p.a_off + r], z);
+    }
     al[d] = expf(log_sigmoid_f(z) / p.tau);
-    ks[d] = row[p.k_off + ch];
-    qs[d] = row[p.q_off + ch] * qscale;
+    ks[d] = k;
+    qs[d] = q * qscale;
   }
   __syncthreads();
-  float4* st = reinterpret_cast<float4*>(p.state) + ((size_t)b * p.H + h) * p.dim * quads;
-  const float* vrow = row + p.v_off + h * p.vdim;
   for (int base = 0; base < cn; base += kGdThreads) {
     const int cols = min(cn - base, kGdThreads), groups = kGdThreads / cols, gi = tid / cols, c = tid - gi * cols;
     float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (gi < groups) {
+    auto advance = [&](float4 s, const float4& vv, int d) {
+      const float a = al[d], k = ks[d], q = qs[d];
+      s.x = fmaf(s.x, a, k * vv.x); s.y = fmaf(s.y, a, k * vv.y); s.z = fmaf(s.z, a, k * vv.z); s.w = fmaf(s.w, a, k * vv.w);
+      st[(size_t)d * quads + c0 + base + c] = s;
+      o.x = fmaf(s.x, q, o.x); o.y = fmaf(s.y, q, o.y); o.z = fmaf(s.z, q, o.z); o.w = fmaf(s.w, q, o.w);
+    };
+    if (pre) {
+#pragma unroll
+      for (int i = 0; i < kGdPre; ++i) {
+        const int d = g0 + i * groups0;
+        if (g0 < groups0 && d < p.dim) advance(sreg[i], vpre, d);
+      }
+    } else if (gi < groups) {
       const int v = 4 * (c0 + base + c);
       const float4 vv = make_float4(v < p.vdim ? vrow[v] : 0.f, v + 1 < p.vdim ? vrow[v + 1] : 0.f, v + 2 < p.vdim ? vrow[v + 2] : 0.f,
                                     v + 3 < p.vdim ? vrow[v + 3] : 0.f);
-#pragma unroll 8
-      for (int d = gi; d < p.dim; d += groups) {
-        float4* sp = st + (size_t)d * quads + c0 + base + c;
-        float4 s = *sp;
-        const float a = al[d], k = ks[d], q = qs[d];
-        s.x = fmaf(s.x, a, k * vv.x); s.y = fmaf(s.y, a, k * vv.y); s.z = fmaf(s.z, a, k * vv.z); s.w = fmaf(s.w, a, k * vv.w);
-        *sp = s;
-        o.x = fmaf(s.x, q, o.x); o.y = fmaf(s.y, q, o.y); o.z = fmaf(s.z, q, o.z); o.w = fmaf(s.w, q, o.w);
-      }
+#pragma unroll 4
+      for (int d = gi; d < p.dim; d += groups) advance(st[(size_t)d * quads + c0 + base + c], vv, d);
     }
     part[tid] = o;
     __syncthreads();
@@ -376,6 +758,31 @@ template <typename T> static int gla_prefill(const nb_gla_args& a, const GlaWs& 
   return check_launch();
 }
 
+// bf16 projections with vdim <= VD: decay, state, scan and output kernels, the last with the norm and the gate.
+template <int VD> static int gla_prefill_mma(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
+  const int chunks = gla_chunks(a.T), subs = (a.T + kGS - 1) / kGS, dt = (a.dim + 63) / 64, HD = a.H * a.dim;
+  const int vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ldp % 8 == 0 && a.q_off % 8 == 0 && a.k_off % 8 == 0 && a.v_off % 8 == 0 &&
+                  a.g_off % 2 == 0 && a.ldo % 2 == 0 && (uintptr_t)a.p % 16 == 0 && (uintptr_t)a.out % 4 == 0;
+  static bool done[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!done[dev & 63]) {
+    if (cudaError_t e = cudaFuncSetAttribute(gla_state_mma_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaStateSmem<VD>)))
+      return record_cuda_error(e);
+    if (cudaError_t e = cudaFuncSetAttribute(gla_output_mma_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaOutSmem<VD>)))
+      return record_cuda_error(e);
+    done[dev & 63] = true;
+  }
+  gla_decay_kernel<bf16><<<dim3(subs, (HD + kDecThreads - 1) / kDecThreads, a.B), kDecThreads, (size_t)kGS * a.a_rank * 4, st>>>(a, w);
+  if (int rc = check_launch()) return rc;
+  gla_state_mma_kernel<VD><<<dim3(chunks, a.H * dt, a.B), kGmThreads, sizeof(GlaStateSmem<VD>), st>>>(a, w, dt, vec);
+  if (int rc = check_launch()) return rc;
+  gla_scan_kernel<<<dim3((a.dim * (a.lds / 4) + 255) / 256, a.B * a.H), 256, 0, st>>>(a, w, chunks);
+  if (int rc = check_launch()) return rc;
+  gla_output_mma_kernel<VD><<<dim3(chunks, a.H, a.B), kGmThreads, sizeof(GlaOutSmem<VD>), st>>>(a, w, vec);
+  return check_launch();
+}
+
 static int gla_check(const nb_gla_args* a) {
   if (!a || !a->p || !a->out || !a->state || !a->a2 || !a->a2_b || !a->norm_w || a->B < 1 || a->T < 1 || a->H < 1 || a->dim < 1 || a->vdim < 1 ||
       a->a_rank < 1 || !(a->tau > 0.f))
@@ -386,7 +793,7 @@ static int gla_check(const nb_gla_args* a) {
       a->v_off + hv > a->ldp || a->g_off + hv > a->ldp || a->a_off + a->a_rank > a->ldp || a->lda2 < a->a_rank || a->ldo < hv ||
       a->lds < a->vdim || a->lds % 4 || a->H > 65535 || a->B > 65535 || (long long)a->B * a->H > 65535)
     return NB_ERR_SHAPE;
-  if ((uintptr_t)a->state % 16) return NB_ERR_ALIGN;
+  if ((uintptr_t)a->state % 16 || (uintptr_t)a->a2 % 16 || a->lda2 % 8) return NB_ERR_ALIGN;
   return NB_OK;
 }
 
@@ -421,7 +828,12 @@ extern "C" int nb_gla_prefill(const nb_gla_args* a, void* workspace, size_t work
   w.dec = reinterpret_cast<float*>(base);
   base += round256(ch * a->dim * 4);
   w.o = reinterpret_cast<float*>(base);
-  return a->dtype == NB_BF16 ? gla_prefill<bf16>(*a, w, (cudaStream_t)stream) : gla_prefill<float>(*a, w, (cudaStream_t)stream);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (a->dtype == NB_F32) return gla_prefill<float>(*a, w, st);
+  return a->vdim <= 64    ? gla_prefill_mma<64>(*a, w, st)
+         : a->vdim <= 128 ? gla_prefill_mma<128>(*a, w, st)
+         : a->vdim <= 256 ? gla_prefill_mma<256>(*a, w, st)
+                          : gla_prefill<bf16>(*a, w, st);
 }
 
 extern "C" int nb_gla_decode(const nb_gla_args* a, void* stream) {

@@ -14,6 +14,7 @@
 #include <cfloat>
 
 #include "nb_layered.cuh"
+#include "nb_mma.cuh"
 
 namespace nb {
 
@@ -50,6 +51,74 @@ template <typename T> __global__ void __launch_bounds__(kPrepThreads) latent_pre
     const float *cs = p.cos2 + (size_t)pos * p.rot, *sn = p.sin2 + (size_t)pos * p.rot;
     for (int d = tid; d < p.rot; d += kPrepThreads)
       c[p.rank + d] = from_f<T>(rotated([&](int i) { return to_f(kv[p.rank + i]); }, cs, sn, d));
+  }
+}
+
+// The same for bf16 rows whose pieces are all multiples of eight: one warp per query latent, one per key/value row, sixteen
+// bytes per lane and load, everything of a row in flight at once and kept in registers between the norm's two passes.
+constexpr int kPvQ = 8;                // loads per lane: up to 2048 columns
+
+template <int N> __device__ __forceinline__ void norm_row_bf16(const bf16* __restrict__ src, const float* __restrict__ w, float eps, int cols,
+                                                               bf16* __restrict__ dst, int lane) {
+  uint4 v[N];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    v[i] = c < cols ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0u, 0u, 0u, 0u);
+  }
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const uint32_t u[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += bf_lo(u[e]) * bf_lo(u[e]) + bf_hi(u[e]) * bf_hi(u[e]);
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)cols + eps);
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const int c = (i * 32 + lane) * 8;
+    if (c < cols) {
+      const uint32_t u[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+      const float4 a = __ldg(reinterpret_cast<const float4*>(w + c)), b = __ldg(reinterpret_cast<const float4*>(w + c + 4));
+      const float wv[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+      uint32_t r[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) r[e] = pack_bf16(bf_lo(u[e]) * inv * wv[2 * e], bf_hi(u[e]) * inv * wv[2 * e + 1]);
+      *reinterpret_cast<uint4*>(dst + c) = make_uint4(r[0], r[1], r[2], r[3]);
+    }
+  }
+}
+
+__global__ void __launch_bounds__(256) latent_prepare_vec_kernel(const nb_latent_prepare_args p, int rows) {
+  pdl_enter();
+  const int lane = threadIdx.x & 31, unit = blockIdx.x * 8 + (threadIdx.x >> 5);
+  const bool is_kv = unit >= rows;
+  const int row = is_kv ? unit - rows : unit;
+  if (row >= rows || (is_kv && p.kv_off < 0)) return;
+  const bf16* a = reinterpret_cast<const bf16*>(p.a) + (size_t)row * p.lda;
+  if (!is_kv) {
+    bf16* cq = reinterpret_cast<bf16*>(p.cq) + (size_t)row * p.ldcq;
+    if (p.q_rank <= 1024) norm_row_bf16<kPvQ / 2>(a + p.q_off, p.q_norm, p.eps, p.q_rank, cq, lane);
+    else norm_row_bf16<kPvQ>(a + p.q_off, p.q_norm, p.eps, p.q_rank, cq, lane);
+    return;
+  }
+  const int b = row / p.T, pos = p.pos0 + row - b * p.T;
+  bf16* c = reinterpret_cast<bf16*>(p.cache) + ((size_t)b * p.ctx + pos) * p.ldc;
+  const bf16* kv = a + p.kv_off;
+  if (p.rank <= 512) norm_row_bf16<2>(kv, p.kv_norm, p.eps, p.rank, c, lane);
+  else norm_row_bf16<kPvQ>(kv, p.kv_norm, p.eps, p.rank, c, lane);
+  for (int d = lane * 8; d < p.rot; d += 256) {
+    const uint4 t = *reinterpret_cast<const uint4*>(kv + p.rank + d);
+    const uint32_t u[4] = {t.x, t.y, t.z, t.w};
+    uint32_t r[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 cs = *reinterpret_cast<const float2*>(p.cos2 + (size_t)pos * p.rot + d + 2 * e);
+      const float2 sn = *reinterpret_cast<const float2*>(p.sin2 + (size_t)pos * p.rot + d + 2 * e);
+      const float x = bf_lo(u[e]), y = bf_hi(u[e]);
+      r[e] = pack_bf16(x * cs.x - y * sn.x, y * cs.y + x * sn.y);
+    }
+    *reinterpret_cast<uint4*>(c + p.rank + d) = make_uint4(r[0], r[1], r[2], r[3]);
   }
 }
 
@@ -158,26 +227,6 @@ __global__ void __launch_bounds__(kLThreads) latent_attention_f32_kernel(const n
 // are not rounded to eight bits.
 constexpr int kTQ = 64, kTK = 64, kTThreads = 128;
 
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)) : "memory");
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<const uint32_t*>(&h);
-}
-
 template <int VD>
 __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const nb_latent_attention_args p, int dk16, int vec) {
   extern __shared__ __align__(16) bf16 tsm[];
@@ -210,18 +259,21 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
     bf16* kd = k_s + st * kTK * dkp;
     bf16* vd = v_s + st * kTK * vp;
     if (vec) {
-      const int nd = p.dim >> 3, nr = p.rot >> 3, nk = nd + nr, nv = p.vdim >> 3;
-      for (int i = tid; i < kTK * (nk + nv); i += kTThreads) {
-        const int j = i / (nk + nv), c = i - j * (nk + nv), pos = k0 + j;
-        bf16* dst = c < nk ? kd + j * dkp + c * 8 : vd + j * vp + (c - nk) * 8;
+      // eight threads per row, 16 bytes each: 128 consecutive bytes of one piece at a time
+      const int c8 = (tid & 7) * 8;
+#pragma unroll
+      for (int jr = 0; jr < kTK; jr += kTThreads / 8) {
+        const int j = jr + (tid >> 3), pos = k0 + j;
+        bf16 *kr = kd + j * dkp, *vr = vd + j * vp;
         if (pos <= last) {
           const bf16* row = kv + (size_t)(pos - p.kv_pos0) * p.ldkv;
-          const bf16* src = c < nd ? row + h * p.dim + c * 8
-                            : c < nk ? cache + (size_t)pos * p.ldc + p.rank + (c - nd) * 8
-                                     : row + p.v_off + h * p.vdim + (c - nk) * 8;
-          cp16(dst, src);
+          const bf16* cr = cache + (size_t)pos * p.ldc + p.rank;
+          for (int c = c8; c < p.dim; c += 64) cp16(kr + c, row + h * p.dim + c);
+          for (int c = c8; c < p.rot; c += 64) cp16(kr + p.dim + c, cr + c);
+          for (int c = c8; c < p.vdim; c += 64) cp16(vr + c, row + p.v_off + h * p.vdim + c);
         } else {
-          *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+          for (int c = c8; c < dk; c += 64) *reinterpret_cast<uint4*>(kr + c) = make_uint4(0u, 0u, 0u, 0u);
+          for (int c = c8; c < p.vdim; c += 64) *reinterpret_cast<uint4*>(vr + c) = make_uint4(0u, 0u, 0u, 0u);
         }
       }
     } else {
@@ -256,6 +308,7 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
   // this lane's two rows of the warp's 16 queries: lane / 4 and lane / 4 + 8
   const int rowa = warp * 16 + (lane >> 2);
   const int pos_a = p.pos0 + min(q0 + rowa, p.T - 1), pos_b = p.pos0 + min(q0 + rowa + 8, p.T - 1);
+  const int wlo = p.pos0 + min(q0 + warp * 16, p.T - 1), whi = p.pos0 + min(q0 + warp * 16 + 15, p.T - 1);   // of the warp's queries
   const float sl2 = p.scale * 1.4426950408889634f;     // softmax in base 2
   float o[VD / 8][4];
 #pragma unroll
@@ -280,6 +333,7 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
     for (int i = 0; i < 8; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
+#pragma unroll 4
     for (int kk = 0; kk < dk16; kk += 16) {
       uint32_t a[4];
       ldsm_x4(a, q_s + (warp * 16 + (lane & 15)) * dkp + kk + (lane >> 4) * 8);
@@ -291,32 +345,39 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
         mma_bf16(s[2 * n + 1], a, bb[2], bb[3]);
       }
     }
+    // a tile that every query of the warp sees whole needs no mask
+    const bool whole = k0 + kTK - 1 <= wlo && (p.window <= 0 || whi - k0 < p.window);
+    if (!whole) {
+#pragma unroll
+      for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int pos = k0 + n * 8 + (lane & 3) * 2 + (j & 1), me = j < 2 ? pos_a : pos_b;
+          if (!(pos <= me && (p.window <= 0 || me - pos < p.window))) s[n][j] = -INFINITY;
+        }
+    }
     float na = ma, nb_ = mb;
 #pragma unroll
-    for (int n = 0; n < 8; ++n)
-#pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const int pos = k0 + n * 8 + (lane & 3) * 2 + (j & 1), me = j < 2 ? pos_a : pos_b;
-        const bool seen = pos <= me && (p.window <= 0 || me - pos < p.window);
-        s[n][j] = seen ? s[n][j] * sl2 : -INFINITY;
-        if (j < 2) na = fmaxf(na, s[n][j]);
-        else nb_ = fmaxf(nb_, s[n][j]);
-      }
+    for (int n = 0; n < 8; ++n) {
+      na = fmaxf(na, fmaxf(s[n][0], s[n][1]));
+      nb_ = fmaxf(nb_, fmaxf(s[n][2], s[n][3]));
+    }
 #pragma unroll
     for (int x = 1; x < 4; x <<= 1) {
       na = fmaxf(na, __shfl_xor_sync(0xffffffffu, na, x));
       nb_ = fmaxf(nb_, __shfl_xor_sync(0xffffffffu, nb_, x));
     }
-    const float ba = na == -INFINITY ? 0.f : na, bb_ = nb_ == -INFINITY ? 0.f : nb_;   // nothing seen yet: all weights are 0
-    const float ca = exp2f(ma - ba), cb = exp2f(mb - bb_);
+    // ma, mb: largest score so far, before the scale (which is positive)
+    const float ba = na == -INFINITY ? 0.f : na * sl2, bb_ = nb_ == -INFINITY ? 0.f : nb_ * sl2;   // nothing seen yet: all weights are 0
+    const float ca = ex2(fmaf(ma, sl2, -ba)), cb = ex2(fmaf(mb, sl2, -bb_));
     ma = na; mb = nb_;
     la *= ca; lb *= cb;
 #pragma unroll
     for (int i = 0; i < VD / 8; ++i) { o[i][0] *= ca; o[i][1] *= ca; o[i][2] *= cb; o[i][3] *= cb; }
 #pragma unroll
     for (int n = 0; n < 8; ++n) {
-      s[n][0] = exp2f(s[n][0] - ba); s[n][1] = exp2f(s[n][1] - ba);
-      s[n][2] = exp2f(s[n][2] - bb_); s[n][3] = exp2f(s[n][3] - bb_);
+      s[n][0] = ex2(fmaf(s[n][0], sl2, -ba)); s[n][1] = ex2(fmaf(s[n][1], sl2, -ba));
+      s[n][2] = ex2(fmaf(s[n][2], sl2, -bb_)); s[n][3] = ex2(fmaf(s[n][3], sl2, -bb_));
       la += s[n][0] + s[n][1];
       lb += s[n][2] + s[n][3];
     }
@@ -326,8 +387,7 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
 #pragma unroll
       for (int j = 0; j < 4; ++j) {                    // registers of the A fragment: (row a, keys 0-7), (row b, ..), (row a, keys 8-15), (row b, ..)
         const float x = s[2 * kk + (j >> 1)][(j & 1) * 2], y = s[2 * kk + (j >> 1)][(j & 1) * 2 + 1];
-        hi[j] = pack_bf16(x, y);
-        lo[j] = pack_bf16(x - bf_lo(hi[j]), y - bf_hi(hi[j]));
+        split_bf16(x, y, hi[j], lo[j]);
       }
 #pragma unroll
       for (int n = 0; n < VD / 16; ++n) {
@@ -368,143 +428,136 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
 
 // ---- one position per sequence.  grid (H, B, S) in clusters of S CTAs along z.  The CTAs of a head share its work three
 // times over: slices of the latent for q' = W_uk^T q, contiguous ranges of the window's keys for the softmax and the
-// weighted latent, slices of the values for W_uv; the slices travel through distributed shared memory.
+// weighted latent, slices of the values for W_uv; the slices travel through distributed shared memory.  A CTA's cached rows
+// are staged in shared memory (`stage` of them at a time, with a running maximum and sum if there are more) and serve as keys
+// and as values from there.  Everything that does not depend on the launch before — the rows of earlier positions, the
+// weights — is requested ahead of the dependency wait.
 constexpr int kLdThreads = 256, kLdWarps = kLdThreads / 32;
+constexpr int kLdCols = 4;             // column pairs per thread: rank <= 2 * 256 * 4
+constexpr int kLdPre = 16;             // W_uk words a thread may hold ahead of the wait
+
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
+template <typename T> __device__ __forceinline__ float dot16(const void* row16, const float* __restrict__ q);
+template <> __device__ __forceinline__ float dot16<bf16>(const void* r, const float* __restrict__ q) {      // eight bf16
+  const uint4 t = *reinterpret_cast<const uint4*>(r);
+  const float4 a = *reinterpret_cast<const float4*>(q), b = *reinterpret_cast<const float4*>(q + 4);
+  return bf_lo(t.x) * a.x + bf_hi(t.x) * a.y + bf_lo(t.y) * a.z + bf_hi(t.y) * a.w + bf_lo(t.z) * b.x + bf_hi(t.z) * b.y + bf_lo(t.w) * b.z +
+         bf_hi(t.w) * b.w;
+}
+template <> __device__ __forceinline__ float dot16<float>(const void* r, const float* __restrict__ q) {     // four fp32
+  const float4 t = *reinterpret_cast<const float4*>(r), a = *reinterpret_cast<const float4*>(q);
+  return t.x * a.x + t.y * a.y + t.z * a.z + t.w * a.w;
+}
+__device__ __forceinline__ float2 pair_at(const bf16* r) {
+  const uint32_t t = *reinterpret_cast<const uint32_t*>(r);
+  return make_float2(bf_lo(t), bf_hi(t));
+}
+__device__ __forceinline__ float2 pair_at(const float* r) { return *reinterpret_cast<const float2*>(r); }
+
+// Elements between staged rows: an odd number of 16-byte pieces, so that eight rows sit on different banks.
+template <typename T> __host__ __device__ inline int staged_row(int rdp) { return rdp % (32 / (int)sizeof(T)) ? rdp : rdp + 16 / (int)sizeof(T); }
 
 template <typename T>
-__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_latent_decode_args p) {
+__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_latent_decode_args p, int stage) {
   extern __shared__ __align__(16) float dsm[];
   __shared__ float red[2 * kLdWarps], red2[kLdWarps], red3[kLdWarps];
   cg::cluster_group cluster = cg::this_cluster();
   const int S = (int)cluster.num_blocks(), rank_id = (int)cluster.block_rank();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int rd = p.rank + p.rot, dk = p.dim + p.rot, rdp = (rd + 7) & ~7;
+  const int rd = p.rank + p.rot, dk = p.dim + p.rot, rdp = (rd + 7) & ~7, ldr = staged_row<T>(rdp);
   float* qa = dsm;                     // [rdp] q' and the rotated query part: what the cached rows are multiplied with
-  float* row = qa + rdp;               // [rdp] this position's row of the cache
-  float* ol = row + rdp;               // [rdp] weighted latent of this CTA's keys, then of all
+  float* ol = qa + rdp;                // [rdp] merged latent
   float* xch = ol + rdp;               // [rdp + 8] what the other CTAs read: weighted latent, maximum, sum
   float* qn = xch + rdp + 8;           // [dk] this head's query
   float* part = qn + ((dk + 7) & ~7);  // [kLdThreads * 2] partial sums
-  float* sc = part + 2 * kLdThreads;   // scores of this CTA's keys
-  pdl_enter();
+  float* sc = part + 2 * kLdThreads;   // [stage] scores, then weights, of the staged keys
+  T* rows = reinterpret_cast<T*>(sc + ((stage + 3) & ~3));   // [stage][ldr]
+
+  // The position was written at the end of the step before, the rows below it in earlier steps or the prompt.
   const long long pos = *p.pos;
   if (pos < 0 || pos >= p.ctx) return; // the same for every CTA
   const int n = p.window > 0 ? min((int)pos + 1, p.window) : (int)pos + 1, first = (int)pos + 1 - n;
   const int per = (n + S - 1) / S, k0 = first + rank_id * per, cnt = max(0, min(first + n, k0 + per) - k0);
   T* cache = reinterpret_cast<T*>(p.cache) + (size_t)b * p.ctx * p.ldc;
+  constexpr int kPiece = 16 / sizeof(T);
+  const int pieces = rdp / kPiece;
+  auto request = [&](int base, int m) {       // rows k0 + base .. of earlier positions
+    for (int j = warp; j < m; j += kLdWarps) {
+      if (k0 + base + j == (int)pos) continue;
+      const T* src = cache + (size_t)(k0 + base + j) * p.ldc;
+      T* dst = rows + (size_t)j * ldr;
+      for (int c = lane; c < pieces; c += 32) cp16(dst + c * kPiece, src + c * kPiece);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  request(0, min(stage, cnt));
+
+  // W_uk: this CTA's slice of columns (pairs), the d range split over groups of threads
+  const int pairs = (p.rank + 1) / 2, pper = (pairs + S - 1) / S, p0 = rank_id * pper, pn = max(0, min(pairs, p0 + pper) - p0);
+  const bf16* uk = reinterpret_cast<const bf16*>(p.uk) + (size_t)h * p.dim * p.ldu;
+  const int cols0 = min(pn, kLdThreads), groups0 = cols0 ? kLdThreads / cols0 : 1, g0 = cols0 ? tid / cols0 : 0, c0 = cols0 ? tid - g0 * cols0 : 0;
+  const bool pre = pn > 0 && pn <= kLdThreads && (p.dim + groups0 - 1) / groups0 <= kLdPre;
+  uint32_t wreg[kLdPre];
+#pragma unroll
+  for (int i = 0; i < kLdPre; ++i) {
+    const int d = g0 + i * groups0;
+    wreg[i] = (pre && g0 < groups0 && d < p.dim) ? __ldg(reinterpret_cast<const uint32_t*>(uk + (size_t)d * p.ldu + 2 * (p0 + c0))) : 0u;
+  }
+  const int vper = (p.vdim + S - 1) / S, v0 = rank_id * vper, v1 = min(p.vdim, v0 + vper);
+  const bf16* uv = reinterpret_cast<const bf16*>(p.uv) + (size_t)h * p.vdim * p.ldu;
+  for (int i = tid; i < (v1 - v0) * ((p.rank + 63) / 64); i += kLdThreads) {
+    const int v = i / ((p.rank + 63) / 64), c = i - v * ((p.rank + 63) / 64);
+    prefetch_l2(uv + (size_t)(v0 + v) * p.ldu + c * 64);
+  }
   const float *cs = p.cos2 + (size_t)pos * p.rot, *sn = p.sin2 + (size_t)pos * p.rot;
 
+  pdl_enter();
   for (int i = tid; i < dk; i += kLdThreads) qn[i] = p.q[(size_t)b * p.ldq + h * dk + i];
-  for (int i = rd + tid; i < rdp; i += kLdThreads) { qa[i] = 0.f; row[i] = 0.f; }
-  if (p.kv_off >= 0) {
-    const float* kv = p.a + (size_t)b * p.lda + p.kv_off;
-    float mean, inv;
+  for (int i = rd + tid; i < rdp; i += kLdThreads) qa[i] = 0.f;
+  // this position's row: from the projection (and written to the cache by one CTA) or from the cache
+  const int mine = (int)pos - k0;      // its place among this CTA's keys, if 0 <= mine < cnt
+  const bool holds = mine >= 0 && mine < cnt;
+  float mean, inv = 0.f;
+  const float* kv = p.a + (size_t)b * p.lda + max(p.kv_off, 0);
+  if (p.kv_off >= 0 && holds)          // block-uniform
     norm_stats<kLdWarps>(NB_NORM_RMS, p.rank, p.eps, red,
                          [&](auto f) { for (int i = tid; i < p.rank; i += kLdThreads) f(kv[i]); }, mean, inv);
+  auto put_row = [&](T* dst) {         // dst: the staged row
     T* crow = cache + (size_t)pos * p.ldc;
-    for (int i = tid; i < rd; i += kLdThreads) {
-      const T v = from_f<T>(i < p.rank ? kv[i] * inv * p.kv_norm[i] : rotated([&](int j) { return kv[p.rank + j]; }, cs, sn, i - p.rank));
-      row[i] = to_f(v);
-      if (h == 0 && rank_id == 0) crow[i] = v;
+    for (int i = tid; i < rdp; i += kLdThreads) {
+      T v = from_f<T>(0.f);
+      if (i < rd) {
+        if (p.kv_off >= 0) {
+          v = from_f<T>(i < p.rank ? kv[i] * inv * p.kv_norm[i] : rotated([&](int j) { return kv[p.rank + j]; }, cs, sn, i - p.rank));
+          if (h == 0) crow[i] = v;
+        } else {
+          v = crow[i];
+        }
+      }
+      dst[i] = v;
     }
-  } else {
-    for (int i = tid; i < rd; i += kLdThreads) row[i] = to_f(cache[(size_t)pos * p.ldc + i]);
-  }
+  };
   cluster.sync();                      // every CTA of the cluster runs: its shared memory may be written from here on
   for (int d = tid; d < p.rot; d += kLdThreads) qa[p.rank + d] = rotated([&](int j) { return qn[p.dim + j]; }, cs, sn, d);
 
-  // q'[j] = sum_d W_uk[h][d][j] q[d] for this CTA's slice of j (pairs), the d range split over groups of threads
-  const int pairs = (p.rank + 1) / 2, pper = (pairs + S - 1) / S, p0 = rank_id * pper, pn = max(0, min(pairs, p0 + pper) - p0);
-  {
-    const bf16* uk = reinterpret_cast<const bf16*>(p.uk) + (size_t)h * p.dim * p.ldu;
-    for (int base = 0; base < pn; base += kLdThreads) {
-      const int cols = min(pn - base, kLdThreads), groups = kLdThreads / cols, gi = tid / cols, c = tid - gi * cols;
-      float x = 0.f, y = 0.f;
-      if (gi < groups) {
-        const int j = 2 * (p0 + base + c);
-#pragma unroll 8
-        for (int d = gi; d < p.dim; d += groups) {
-          const uint32_t w = *reinterpret_cast<const uint32_t*>(uk + (size_t)d * p.ldu + j);
-          x = fmaf(bf_lo(w), qn[d], x);
-          y = fmaf(bf_hi(w), qn[d], y);
-        }
-      }
-      part[2 * tid] = x; part[2 * tid + 1] = y;
-      __syncthreads();
-      for (int i = tid; i < 2 * cols; i += kLdThreads) {
-        float v = 0.f;
-        for (int g = 0; g < groups; ++g) v += part[2 * g * cols + i];
-        const int j = 2 * (p0 + base) + i;
-        if (j < p.rank)
-          for (int r = 0; r < S; ++r) cluster.map_shared_rank(qa, r)[j] = v;
-      }
-      __syncthreads();
-    }
-  }
-  cluster.sync();
-
-  // scores: a warp takes a key at a time, eight columns per lane and step
-  float mx = -FLT_MAX;
-  for (int j = warp; j < cnt; j += kLdWarps) {
-    float s = 0.f;
-    if (k0 + j == (int)pos) {
-      for (int i = lane; i < rd; i += 32) s = fmaf(row[i], qa[i], s);
-    } else {
-      const T* cr = cache + (size_t)(k0 + j) * p.ldc;
-      if (sizeof(T) == 2) {
-        for (int i = lane * 8; i < rd; i += 256) {
-          const uint4 t = *reinterpret_cast<const uint4*>(cr + i);   // ldc is a multiple of 8; past rd qa is zero
-          const float4 a = *reinterpret_cast<const float4*>(qa + i), c = *reinterpret_cast<const float4*>(qa + i + 4);
-          const uint32_t u[4] = {t.x, t.y, t.z, t.w};
-          const float q8[8] = {a.x, a.y, a.z, a.w, c.x, c.y, c.z, c.w};
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            if (i + 2 * e < rd) s = fmaf(bf_lo(u[e]), q8[2 * e], s);
-            if (i + 2 * e + 1 < rd) s = fmaf(bf_hi(u[e]), q8[2 * e + 1], s);
-          }
-        }
-      } else {
-        for (int i = lane; i < rd; i += 32) s = fmaf(to_f(cr[i]), qa[i], s);
-      }
-    }
-    s = warp_sum(s) * p.scale;
-    if (lane == 0) sc[j] = s;
-    mx = fmaxf(mx, s);
-  }
-  if (lane == 0) red2[warp] = mx;
-  __syncthreads();
-  mx = red2[0];
-#pragma unroll
-  for (int i = 1; i < kLdWarps; ++i) mx = fmaxf(mx, red2[i]);
-  float sum = 0.f;
-  for (int j = tid; j < cnt; j += kLdThreads) {
-    const float e = expf(sc[j] - mx);
-    sc[j] = e;
-    sum += e;
-  }
-  const float tot = block_sum<kLdWarps>(sum, red3);    // its barrier also publishes sc
-
-  // weighted latent of this CTA's keys: pairs of columns per thread, the keys split over groups of threads
-  for (int base = 0; base < pairs; base += kLdThreads) {
-    const int cols = min(pairs - base, kLdThreads), groups = kLdThreads / cols, gi = tid / cols, c = tid - gi * cols;
+  // q'[j] = sum_d W_uk[h][d][j] q[d]
+  for (int base = 0; base < pn; base += kLdThreads) {
+    const int cols = min(pn - base, kLdThreads), groups = kLdThreads / cols, gi = tid / cols, c = tid - gi * cols;
     float x = 0.f, y = 0.f;
-    if (gi < groups) {
-      const int i = 2 * (base + c);
-#pragma unroll 4
-      for (int j = gi; j < cnt; j += groups) {
-        const float w = sc[j];
-        if (k0 + j == (int)pos) {
-          x = fmaf(w, row[i], x);
-          y = fmaf(w, row[i + 1], y);
-        } else if (sizeof(T) == 2) {
-          const uint32_t t = *reinterpret_cast<const uint32_t*>(cache + (size_t)(k0 + j) * p.ldc + i);
-          x = fmaf(w, bf_lo(t), x);
-          y = fmaf(w, bf_hi(t), y);
-        } else {
-          const float2 t = *reinterpret_cast<const float2*>(cache + (size_t)(k0 + j) * p.ldc + i);
-          x = fmaf(w, t.x, x);
-          y = fmaf(w, t.y, y);
-        }
+    if (pre) {
+#pragma unroll
+      for (int i = 0; i < kLdPre; ++i) {
+        const int d = g0 + i * groups0;
+        if (d < p.dim) { x = fmaf(bf_lo(wreg[i]), qn[d], x); y = fmaf(bf_hi(wreg[i]), qn[d], y); }
+      }
+    } else if (gi < groups) {
+      const int j = 2 * (p0 + base + c);
+#pragma unroll 8
+      for (int d = gi; d < p.dim; d += groups) {
+        const uint32_t w = *reinterpret_cast<const uint32_t*>(uk + (size_t)d * p.ldu + j);
+        x = fmaf(bf_lo(w), qn[d], x);
+        y = fmaf(bf_hi(w), qn[d], y);
       }
     }
     part[2 * tid] = x; part[2 * tid + 1] = y;
@@ -512,41 +565,121 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
     for (int i = tid; i < 2 * cols; i += kLdThreads) {
       float v = 0.f;
       for (int g = 0; g < groups; ++g) v += part[2 * g * cols + i];
-      xch[2 * base + i] = v;
+      const int j = 2 * (p0 + base) + i;
+      if (j < p.rank)
+        for (int r = 0; r < S; ++r) cluster.map_shared_rank(qa, r)[j] = v;
     }
     __syncthreads();
   }
-  if (tid == 0) { xch[rdp] = mx; xch[rdp + 1] = tot; }
+  cluster.sync();
+
+  // softmax and weighted latent over the staged rows.  Scores: four lanes share a key, sixteen bytes at a time.  Latent: a
+  // thread owns up to kLdCols column pairs, or, with few columns, one pair of every `groups`-th key.
+  const int wcols = min(pairs, kLdThreads), groups = pairs <= kLdThreads ? kLdThreads / wcols : 1, gi = tid / wcols, wc = tid - gi * wcols;
+  float m = -FLT_MAX, l = 0.f;
+  float2 acc[kLdCols];
+#pragma unroll
+  for (int u = 0; u < kLdCols; ++u) acc[u] = make_float2(0.f, 0.f);
+  for (int base = 0; base < cnt; base += stage) {
+    const int nk = min(stage, cnt - base);
+    if (base > 0) {
+      __syncthreads();                 // the rows and weights before are no longer read
+      request(base, nk);
+    }
+    if (mine >= base && mine < base + nk) put_row(rows + (size_t)(mine - base) * ldr);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    float mx = -FLT_MAX;
+    for (int j0 = warp * 8; j0 < nk; j0 += kLdWarps * 8) {
+      const int j = j0 + (lane >> 2);
+      float s = 0.f;
+      if (j < nk) {
+        const T* r = rows + (size_t)j * ldr;
+        for (int c = lane & 3; c < pieces; c += 4) s += dot16<T>(r + c * kPiece, qa + c * kPiece);
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      s *= p.scale;
+      if (j < nk) {
+        if ((lane & 3) == 0) sc[j] = s;
+        mx = fmaxf(mx, s);
+      }
+    }
+    mx = warp_max(mx);
+    if (lane == 0) red2[warp] = mx;
+    __syncthreads();
+    float m_new = m;
+#pragma unroll
+    for (int i = 0; i < kLdWarps; ++i) m_new = fmaxf(m_new, red2[i]);
+    const float corr = expf(m - m_new);
+    m = m_new;
+    float sum = 0.f;
+    for (int j = tid; j < nk; j += kLdThreads) {
+      const float e = expf(sc[j] - m);
+      sc[j] = e;
+      sum += e;
+    }
+    l = l * corr + block_sum<kLdWarps>(sum, red3);   // its barrier also publishes the weights
+#pragma unroll
+    for (int u = 0; u < kLdCols; ++u) {
+      acc[u].x *= corr; acc[u].y *= corr;
+      const int c = wc + u * kLdThreads;
+      if (gi < groups && c < pairs) {
+#pragma unroll 8
+        for (int j = gi; j < nk; j += groups) {
+          const float w = sc[j];
+          const float2 t = pair_at(rows + (size_t)j * ldr + 2 * c);
+          acc[u].x = fmaf(w, t.x, acc[u].x);
+          acc[u].y = fmaf(w, t.y, acc[u].y);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < kLdCols; ++u) {
+    if (u * kLdThreads < pairs) {      // block-uniform
+      part[2 * tid] = acc[u].x; part[2 * tid + 1] = acc[u].y;
+      __syncthreads();
+      const int cols = min(pairs - u * kLdThreads, kLdThreads);
+      for (int i = tid; i < 2 * cols; i += kLdThreads) {
+        float v = 0.f;
+        for (int g = 0; g < groups; ++g) v += part[2 * g * wcols + i];
+        xch[2 * u * kLdThreads + i] = v;
+      }
+      __syncthreads();
+    }
+  }
+  if (tid == 0) { xch[rdp] = m; xch[rdp + 1] = l; }
   cluster.sync();
   // this CTA's slice of the merged latent, to everyone
   {
-    float m_all = -FLT_MAX, den = 0.f;
+    float m_all = -FLT_MAX, den = 0.f, wr[8];
     for (int r = 0; r < S; ++r) m_all = fmaxf(m_all, cluster.map_shared_rank(xch, r)[rdp]);
-    for (int r = 0; r < S; ++r) {      // a CTA without keys has maximum -FLT_MAX and sum 0
-      const float* rx = cluster.map_shared_rank(xch, r);
-      den += expf(rx[rdp] - m_all) * rx[rdp + 1];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {      // a CTA without keys has maximum -FLT_MAX and sum 0
+      wr[r] = 0.f;
+      if (r < S) {
+        const float* rx = cluster.map_shared_rank(xch, r);
+        wr[r] = expf(rx[rdp] - m_all);
+        den += wr[r] * rx[rdp + 1];
+      }
     }
     for (int i = 2 * p0 + tid; i < min(p.rank, 2 * (p0 + pn)); i += kLdThreads) {
       float num = 0.f;
-      for (int r = 0; r < S; ++r) {
-        const float* rx = cluster.map_shared_rank(xch, r);
-        num += expf(rx[rdp] - m_all) * rx[i];
-      }
+#pragma unroll
+      for (int r = 0; r < 8; ++r)
+        if (r < S) num += wr[r] * cluster.map_shared_rank(xch, r)[i];
       const float v = num / den;
       for (int r = 0; r < S; ++r) cluster.map_shared_rank(ol, r)[i] = v;
     }
   }
+  for (int i = p.rank + tid; i < ((p.rank + 7) & ~7); i += kLdThreads) ol[i] = 0.f;   // W_uv is read in eights
   cluster.sync();                      // also: nobody reads another CTA's shared memory after this
-  const int vper = (p.vdim + S - 1) / S, v0 = rank_id * vper, v1 = min(p.vdim, v0 + vper);
   const float g = sigmoid_f(p.a[(size_t)b * p.lda + p.g_off + h]);
   for (int v = v0 + warp; v < v1; v += kLdWarps) {
-    const bf16* uv = reinterpret_cast<const bf16*>(p.uv) + (size_t)(h * p.vdim + v) * p.ldu;
+    const bf16* wv = uv + (size_t)v * p.ldu;
     float s = 0.f;
-    for (int i = lane * 2; i < p.rank; i += 64) {
-      const uint32_t w = *reinterpret_cast<const uint32_t*>(uv + i);
-      s = fmaf(bf_lo(w), ol[i], s);
-      if (i + 1 < p.rank) s = fmaf(bf_hi(w), ol[i + 1], s);
-    }
+    for (int i = lane * 8; i < p.rank; i += 256) s += dot16<bf16>(wv + i, ol + i);
     s = warp_sum(s);
     if (lane == 0) p.out[(size_t)b * p.ldo + h * p.vdim + v] = s * g;
   }
@@ -603,13 +736,23 @@ extern "C" int nb_latent_prepare(const nb_latent_prepare_args* a, void* stream) 
   }
   if (int rc = check_device()) return rc;
   const dim3 grid((unsigned)a->B * a->T);
+  const bool kv = a->kv_off >= 0;
+  const bool vec = a->dtype == NB_BF16 && a->q_rank % 8 == 0 && a->q_off % 8 == 0 && a->lda % 8 == 0 && a->ldcq % 8 == 0 &&
+                   a->q_rank <= 256 * kPvQ && (uintptr_t)a->a % 16 == 0 && (uintptr_t)a->cq % 16 == 0 && (uintptr_t)a->q_norm % 16 == 0 &&
+                   (!kv || (a->kv_off % 8 == 0 && a->rank % 8 == 0 && a->rot % 8 == 0 && a->rank <= 256 * kPvQ && a->ldc % 8 == 0 &&
+                            (uintptr_t)a->cache % 16 == 0 && (uintptr_t)a->kv_norm % 16 == 0 && (uintptr_t)a->cos2 % 8 == 0 &&
+                            (uintptr_t)a->sin2 % 8 == 0));
+  if (vec) {
+    const int rows = a->B * a->T;
+    return launch_pdl(latent_prepare_vec_kernel, dim3(((kv ? 2 : 1) * rows + 7) / 8), dim3(256), 0, (cudaStream_t)stream, *a, rows);
+  }
   return a->dtype == NB_BF16 ? launch_pdl(latent_prepare_kernel<bf16>, grid, dim3(kPrepThreads), 0, (cudaStream_t)stream, *a)
                              : launch_pdl(latent_prepare_kernel<float>, grid, dim3(kPrepThreads), 0, (cudaStream_t)stream, *a);
 }
 
 extern "C" int nb_latent_attention(const nb_latent_attention_args* a, void* stream) {
   if (!a || !a->q || !a->kv || !a->cache || !a->out || !a->cos2 || !a->sin2 || a->B < 1 || a->T < 1 || a->H < 1 || a->dim < 1 || a->rot < 0 ||
-      a->rot % 2 || a->vdim < 1 || a->pos0 < 0 || a->window < 0 || a->kv_pos0 < 0)
+      a->rot % 2 || a->vdim < 1 || a->pos0 < 0 || a->window < 0 || a->kv_pos0 < 0 || !(a->scale > 0.f))
     return NB_ERR_ARG;
   if (a->dtype != NB_BF16 && a->dtype != NB_F32) return NB_ERR_ARG;
   const int first = a->window > 0 ? std::max(0, a->pos0 - a->window + 1) : 0;
@@ -638,18 +781,23 @@ extern "C" int nb_latent_decode(const nb_latent_decode_args* a, void* stream) {
   if ((uintptr_t)a->cache % 16 || a->ldc % 8 || (uintptr_t)a->uk % 16 || (uintptr_t)a->uv % 16 || a->ldu % 8) return NB_ERR_ALIGN;
   if (a->H > 65535 || a->B > 65535) return NB_ERR_SHAPE;
   if (int rc = check_device()) return rc;
+  if (a->rank > 2 * kLdThreads * kLdCols) return NB_ERR_SHAPE;
   const int want = 592 / std::max(1, a->B * a->H), S = want >= 8 ? 8 : want >= 4 ? 4 : want >= 2 ? 2 : 1;
   const int most = a->window > 0 ? std::min(a->window, a->ctx) : a->ctx;
+  const int wide = a->cache_dtype == NB_F32;
   const int rdp = (a->rank + a->rot + 7) & ~7;
-  const size_t smem = ((size_t)4 * rdp + 8 + ((a->dim + a->rot + 7) & ~7) + 2 * kLdThreads + (most + S - 1) / S + 8) * 4;
-  if (smem > kLatentMaxSmem) return NB_ERR_SHAPE;
+  const size_t row = (size_t)(wide ? staged_row<float>(rdp) * 4 : staged_row<bf16>(rdp) * 2);
+  const size_t fixed = ((size_t)3 * rdp + 8 + ((a->dim + a->rot + 7) & ~7) + 2 * kLdThreads + 4) * 4;
+  if (fixed + 8 * (row + 4) > kLatentMaxSmem) return NB_ERR_SHAPE;
+  // as many of a CTA's rows at a time as shared memory holds
+  const int stage = (int)std::min<size_t>((most + S - 1) / S, (kLatentMaxSmem - fixed) / (row + 4));
+  const size_t smem = fixed + (size_t)((stage + 3) & ~3) * 4 + stage * row;
   static bool done[2][64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  const int wide = a->cache_dtype == NB_F32;
   auto kernel = wide ? latent_decode_kernel<float> : latent_decode_kernel<bf16>;
   if (!done[wide][dev & 63]) {
-    if (cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentMaxSmem)) return record_cuda_error(e);
+    if (cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kLatentMaxSmem + 64)) return record_cuda_error(e);
     done[wide][dev & 63] = true;
   }
   cudaLaunchConfig_t cfg = {};
@@ -666,5 +814,5 @@ extern "C" int nb_latent_decode(const nb_latent_decode_args* a, void* stream) {
   attr[1].val.clusterDim.z = S;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  return record_cuda_error(cudaLaunchKernelEx(&cfg, kernel, *a));
+  return record_cuda_error(cudaLaunchKernelEx(&cfg, kernel, *a, stage));
 }

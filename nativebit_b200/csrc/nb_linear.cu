@@ -53,6 +53,88 @@ __global__ void __launch_bounds__(kChainThreads) residual_norm_kernel(float* __r
   }
 }
 
+// The same with the row in registers, four values per thread and load: C <= 1024 * NV, a multiple of 4.
+__device__ __forceinline__ void store4(float* p, float a, float b, float c, float d) { *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d); }
+__device__ __forceinline__ void store4(bf16* p, float a, float b, float c, float d) {
+  const __nv_bfloat162 x = __floats2bfloat162_rn(a, b), y = __floats2bfloat162_rn(c, d);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&x), *reinterpret_cast<const uint32_t*>(&y));
+}
+
+// Statistics of a row held as NV float4 per thread (zero past the row's end, `in(i)` tells which are inside).
+template <int kWarps, int NV, typename In>
+__device__ __forceinline__ void norm_stats4(int kind, int C, float eps, float* red, const float4 (&v)[NV], In in, float& mean, float& inv) {
+  mean = 0.f;
+  if (kind == NB_NORM_LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+    mean = block_sum<kWarps>(s, red) / (float)C;
+  }
+  float q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (in(i)) {
+      const float a = v[i].x - mean, b = v[i].y - mean, c = v[i].z - mean, d = v[i].w - mean;
+      q += (a * a + b * b) + (c * c + d * d);
+    }
+  inv = 1.0f / sqrtf(block_sum<kWarps>(q, red + kWarps) / (float)C + eps);
+}
+
+template <typename TH, int NV>
+__global__ void __launch_bounds__(kChainThreads) residual_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ y,
+                                                                          const float* __restrict__ wy, const float* __restrict__ w, int kind,
+                                                                          float eps, TH* __restrict__ h, int ldh, int C) {
+  __shared__ float red[4 * kChainWarps];
+  pdl_enter();
+  const int tid = threadIdx.x;
+  float* xr = x + (size_t)blockIdx.x * C;
+  const float* yr = y ? y + (size_t)blockIdx.x * C : nullptr;
+  auto at = [&](int i) { return (i * kChainThreads + tid) * 4; };
+  auto in = [&](int i) { return at(i) < C; };
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  float4 v[NV];
+  float mean, inv;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) v[i] = in(i) ? *reinterpret_cast<const float4*>(xr + at(i)) : zero;
+  if (yr) {
+    float4 d[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) d[i] = in(i) ? *reinterpret_cast<const float4*>(yr + at(i)) : zero;
+    norm_stats4<kChainWarps, NV>(kind, C, eps, red, d, in, mean, inv);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (in(i)) {
+        const float4 g = __ldg(reinterpret_cast<const float4*>(wy + at(i)));
+        v[i].x += (d[i].x - mean) * inv * g.x; v[i].y += (d[i].y - mean) * inv * g.y;
+        v[i].z += (d[i].z - mean) * inv * g.z; v[i].w += (d[i].w - mean) * inv * g.w;
+        *reinterpret_cast<float4*>(xr + at(i)) = v[i];
+      }
+  }
+  if (h) {
+    norm_stats4<kChainWarps, NV>(kind, C, eps, red + 2 * kChainWarps, v, in, mean, inv);
+    TH* hr = h + (size_t)blockIdx.x * ldh;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (in(i)) {
+        const float4 g = __ldg(reinterpret_cast<const float4*>(w + at(i)));
+        store4(hr + at(i), (v[i].x - mean) * inv * g.x, (v[i].y - mean) * inv * g.y, (v[i].z - mean) * inv * g.z, (v[i].w - mean) * inv * g.w);
+      }
+  }
+}
+
+template <typename TH>
+static int launch_residual_norm(float* x, const float* y, const float* wy, const float* w, int norm, float eps, TH* h, int ldh, int rows, int C,
+                                cudaStream_t st) {
+  const dim3 grid(rows), block(kChainThreads);
+  const bool vec = C % 4 == 0 && ldh % 4 == 0 && C <= 8 * 1024 && (uintptr_t)x % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)wy % 16 == 0 &&
+                   (uintptr_t)w % 16 == 0 && (uintptr_t)h % 16 == 0;
+  if (!vec) return launch_pdl(residual_norm_kernel<TH>, grid, block, (size_t)C * 4, st, x, y, wy, w, norm, eps, h, ldh, C);
+  if (C <= 1024) return launch_pdl(residual_norm_vec_kernel<TH, 1>, grid, block, 0, st, x, y, wy, w, norm, eps, h, ldh, C);
+  if (C <= 2048) return launch_pdl(residual_norm_vec_kernel<TH, 2>, grid, block, 0, st, x, y, wy, w, norm, eps, h, ldh, C);
+  if (C <= 4096) return launch_pdl(residual_norm_vec_kernel<TH, 4>, grid, block, 0, st, x, y, wy, w, norm, eps, h, ldh, C);
+  return launch_pdl(residual_norm_vec_kernel<TH, 8>, grid, block, 0, st, x, y, wy, w, norm, eps, h, ldh, C);
+}
+
 // ---- fp32 product: 64 x 64 output tile per CTA, 16 x 16 threads with 4 x 4 outputs each, k in steps of 16.
 constexpr int kFT = 64, kFKS = 16;
 
@@ -106,8 +188,9 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 // bytes, 16 per lane), is dealt to the CTA's warps in equal contiguous runs, so every SM and every warp streams the
 // same number of bytes whatever N and K are.  A row that lies in one run is finished by its warp; the parts of a row
 // that runs share are added in warp order after a barrier: no atomics, bit-identical from run to run.  Each warp keeps
-// 8 - 16 items in flight in registers and requests the first ones before the dependency wait.
-constexpr int kMvWarps = 16, kMvThreads = kMvWarps * 32, kMvBatch = 8;
+// 8 - 16 items in flight in registers and requests the first ones before the dependency wait; a CTA is small enough
+// that the next launch's CTA fits beside it and starts its own requests while this one drains.
+constexpr int kMvWarps = 8, kMvThreads = kMvWarps * 32, kMvBatch = 8;
 
 struct MatvecParams {
   const uint4* w;
@@ -124,7 +207,8 @@ __device__ __forceinline__ uint4 ld_stream(const uint4* p) {
   return v;
 }
 
-__global__ void __launch_bounds__(kMvThreads, 1) matvec_kernel(const MatvecParams p) {
+template <int NV>   // float4 of the row per thread in the prologue (K <= 1024 * NV, a multiple of 4), 0: any K
+__global__ void __launch_bounds__(kMvThreads, 2) matvec_kernel(const MatvecParams p) {
   extern __shared__ __align__(16) float mv_smem[];
   __shared__ float red[4 * kMvWarps], part_v[2 * kMvWarps];
   __shared__ int part_r[2 * kMvWarps];
@@ -156,28 +240,66 @@ __global__ void __launch_bounds__(kMvThreads, 1) matvec_kernel(const MatvecParam
   for (int r = tid; r < R; r += kMvThreads) ysum[r] = 0.f;
   if (tid < 2 * kMvWarps) part_r[tid] = -1;
 
-  pdl_enter();
-
   auto slot = [](int k) { return (k & ~255) + ((k & 4) << 5) + ((k & 255) >> 3) * 4 + (k & 3); };
-  auto each = [&](auto f) {
-    for (int k = tid; k < p.K; k += kMvThreads) f(xs[slot(k)]);
-  };
-  for (int k = p.K + tid; k < KC * 256; k += kMvThreads) xs[slot(k)] = 0.f;
   float mean, inv;
-  if (p.delta) {
-    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.delta[k];
-    norm_stats<kMvWarps>(p.norm, p.K, p.eps, red, each, mean, inv);
-    for (int k = tid; k < p.K; k += kMvThreads) {
-      const float v = p.x[k] + (xs[slot(k)] - mean) * inv * p.delta_w[k];
-      if (blockIdx.x == 0) p.x_out[k] = v;
-      xs[slot(k)] = v;
+  if constexpr (NV > 0) {
+    // weights of the norms ahead of the wait, the vectors all at once behind it
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    auto at = [&](int i) { return (i * kMvThreads + tid) * 4; };
+    auto in = [&](int i) { return at(i) < p.K; };
+    float4 nw[NV], dw[NV], v[NV], d[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      nw[i] = (p.norm_w && in(i)) ? __ldg(reinterpret_cast<const float4*>(p.norm_w + at(i))) : zero;
+      dw[i] = (p.delta && in(i)) ? __ldg(reinterpret_cast<const float4*>(p.delta_w + at(i))) : zero;
     }
+    pdl_enter();
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      v[i] = in(i) ? *reinterpret_cast<const float4*>(p.x + at(i)) : zero;
+      d[i] = (p.delta && in(i)) ? *reinterpret_cast<const float4*>(p.delta + at(i)) : zero;
+    }
+    if (p.delta) {
+      norm_stats4<kMvWarps, NV>(p.norm, p.K, p.eps, red, d, in, mean, inv);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (in(i)) {
+          v[i].x += (d[i].x - mean) * inv * dw[i].x; v[i].y += (d[i].y - mean) * inv * dw[i].y;
+          v[i].z += (d[i].z - mean) * inv * dw[i].z; v[i].w += (d[i].w - mean) * inv * dw[i].w;
+          if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.x_out + at(i)) = v[i];
+        }
+    }
+    if (p.norm_w) {
+      norm_stats4<kMvWarps, NV>(p.norm, p.K, p.eps, red + 2 * kMvWarps, v, in, mean, inv);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        v[i] = make_float4((v[i].x - mean) * inv * nw[i].x, (v[i].y - mean) * inv * nw[i].y, (v[i].z - mean) * inv * nw[i].z,
+                           (v[i].w - mean) * inv * nw[i].w);
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (at(i) < KC * 256) *reinterpret_cast<float4*>(xs + slot(at(i))) = in(i) ? v[i] : zero;
   } else {
-    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.x[k];
-  }
-  if (p.norm_w) {
-    norm_stats<kMvWarps>(p.norm, p.K, p.eps, red + 2 * kMvWarps, each, mean, inv);
-    for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = (xs[slot(k)] - mean) * inv * p.norm_w[k];
+    pdl_enter();
+    auto each = [&](auto f) {
+      for (int k = tid; k < p.K; k += kMvThreads) f(xs[slot(k)]);
+    };
+    for (int k = p.K + tid; k < KC * 256; k += kMvThreads) xs[slot(k)] = 0.f;
+    if (p.delta) {
+      for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.delta[k];
+      norm_stats<kMvWarps>(p.norm, p.K, p.eps, red, each, mean, inv);
+      for (int k = tid; k < p.K; k += kMvThreads) {
+        const float v = p.x[k] + (xs[slot(k)] - mean) * inv * p.delta_w[k];
+        if (blockIdx.x == 0) p.x_out[k] = v;
+        xs[slot(k)] = v;
+      }
+    } else {
+      for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = p.x[k];
+    }
+    if (p.norm_w) {
+      norm_stats<kMvWarps>(p.norm, p.K, p.eps, red + 2 * kMvWarps, each, mean, inv);
+      for (int k = tid; k < p.K; k += kMvThreads) xs[slot(k)] = (xs[slot(k)] - mean) * inv * p.norm_w[k];
+    }
   }
   __syncthreads();
 
@@ -235,6 +357,19 @@ __global__ void __launch_bounds__(kMvThreads, 1) matvec_kernel(const MatvecParam
   }
 }
 
+constexpr size_t kMvMaxSmem = 200 * 1024;
+
+template <int NV> static int launch_matvec(const MatvecParams& p, int G, size_t smem, cudaStream_t st) {
+  static bool done[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (!done[dev & 63]) {
+    if (cudaError_t e = cudaFuncSetAttribute(matvec_kernel<NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMvMaxSmem)) return record_cuda_error(e);
+    done[dev & 63] = true;
+  }
+  return launch_pdl(matvec_kernel<NV>, dim3(G), dim3(kMvThreads), smem, st, p);
+}
+
 }  // namespace nb
 
 using namespace nb;
@@ -252,12 +387,9 @@ extern "C" int nb_residual_norm(float* x, const float* y, const float* wy, const
   if ((norm != NB_NORM_RMS && norm != NB_NORM_LAYER) || (h_dtype != NB_BF16 && h_dtype != NB_F32)) return NB_ERR_ARG;
   if (C > 12 * 1024) return NB_ERR_SHAPE;   // the row sits in shared memory
   if (int rc = check_device()) return rc;
-  const size_t smem = (size_t)C * 4;
-  if (h_dtype == NB_BF16)
-    return launch_pdl(residual_norm_kernel<bf16>, dim3(rows), dim3(kChainThreads), smem, (cudaStream_t)stream, x, y, wy, w, norm, eps,
-                      reinterpret_cast<bf16*>(h), ldh, C);
-  return launch_pdl(residual_norm_kernel<float>, dim3(rows), dim3(kChainThreads), smem, (cudaStream_t)stream, x, y, wy, w, norm, eps,
-                    reinterpret_cast<float*>(h), ldh, C);
+  return h_dtype == NB_BF16
+             ? launch_residual_norm(x, y, wy, w, norm, eps, reinterpret_cast<bf16*>(h), ldh, rows, C, (cudaStream_t)stream)
+             : launch_residual_norm(x, y, wy, w, norm, eps, reinterpret_cast<float*>(h), ldh, rows, C, (cudaStream_t)stream);
 }
 
 extern "C" int nb_linear_f32(const float* x, int ldx, const void* w, int ldw, const float* bias, int act, int M, int N, int K, float* y,
@@ -285,20 +417,19 @@ extern "C" int nb_matvec_bf16(const nb_matvec_args* a, void* stream) {
   const int G = std::min(sm_count(), a->N / unit);
   const int rows = ((a->N / unit + G - 1) / G) * unit, kc = (a->K + 255) / 256;
   const size_t smem = ((size_t)kc * 256 + rows) * 4;
-  constexpr size_t kMax = 200 * 1024;
-  if (smem > kMax) return NB_ERR_SHAPE;
-  static bool attr_done[64] = {};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (!attr_done[dev & 63]) {
-    if (cudaError_t e = cudaFuncSetAttribute(matvec_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMax)) return record_cuda_error(e);
-    attr_done[dev & 63] = true;
-  }
+  if (smem > kMvMaxSmem) return NB_ERR_SHAPE;
   MatvecParams p;
   p.w = reinterpret_cast<const uint4*>(a->w);
   p.bias = a->bias; p.x = a->x; p.delta = a->delta; p.delta_w = a->delta_w; p.norm_w = a->norm_w;
   p.y = a->y; p.x_out = a->x_out;
   p.eps = a->eps; p.N = a->N; p.K = a->K; p.ldw8 = a->ldw / 8;
   p.act = (short)a->act; p.norm = (short)a->norm;
-  return launch_pdl(matvec_kernel, dim3(G), dim3(kMvThreads), smem, (cudaStream_t)stream, p);
+  const cudaStream_t st = (cudaStream_t)stream;
+  const bool vec = a->K % 4 == 0 && (uintptr_t)a->x % 16 == 0 && (uintptr_t)a->delta % 16 == 0 && (uintptr_t)a->delta_w % 16 == 0 &&
+                   (uintptr_t)a->norm_w % 16 == 0 && (uintptr_t)a->x_out % 16 == 0;
+  if (vec && a->K <= 1024) return launch_matvec<1>(p, G, smem, st);
+  if (vec && a->K <= 2048) return launch_matvec<2>(p, G, smem, st);
+  if (vec && a->K <= 3072) return launch_matvec<3>(p, G, smem, st);
+  if (vec && a->K <= 4096) return launch_matvec<4>(p, G, smem, st);
+  return launch_matvec<0>(p, G, smem, st);
 }
