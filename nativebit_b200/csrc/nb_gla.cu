@@ -54,10 +54,12 @@ template <typename T> __global__ void __launch_bounds__(kDecThreads) gla_decay_k
     for (int t = 0; t < kGS; ++t) z[t] = fmaf(x, as[t * p.a_rank + r], z[t]);
   }
   float sum = 0.f;
+  const float inv_tau = 1.0f / p.tau;
   float* out = w.bl + (size_t)(b * p.T + t0) * HD + ch;
 #pragma unroll
   for (int t = 0; t < kGS; ++t) {
-    sum += log_sigmoid_f(z[t]) / p.tau;
+    // with bf16 projections log(1 + e^-|z|) goes through the hardware functions: absolute errors of 1e-7
+    sum += (sizeof(T) == 2 ? fminf(z[t], 0.f) - __logf(1.f + __expf(-fabsf(z[t]))) : log_sigmoid_f(z[t])) * inv_tau;
     if (t < cnt) out[(size_t)t * HD] = sum;
   }
 }
@@ -293,29 +295,65 @@ template <typename T> __global__ void __launch_bounds__(256) gla_finish_kernel(c
 // product of two such pairs as three).  Four warps per CTA; vdim <= VD.
 constexpr int kGmThreads = 128;
 constexpr int kGmLd = 64 + 8;          // row stride of a staged tile of 64 channels, in elements
+constexpr int kGbLd = 64 + 4;          // row stride of staged log decays
 constexpr float kSplitLimit = -60.f;   // a sub-block that decays further is taken pair by pair
 
 template <int VD> struct GlaStateSmem {
-  bf16 khi[kGC * kGmLd], klo[kGC * kGmLd], v[kGC * (VD + 8)];
-  float tot[kGSubs * 64];
+  bf16 k[kGC * kGmLd], khi[kGC * kGmLd], klo[kGC * kGmLd], v[kGC * (VD + 8)];
+  float bl[kGC * kGbLd], tot[kGSubs * 64];
 };
 
-// Copies rows of `cols` bf16 (zero past `valid` columns and `cnt` rows) into shared memory; vec: 16-byte aligned, cols % 8 == 0.
+// Copies rows of `cols` bf16 (zero past `valid` columns and `cnt` rows) into shared memory; vec: 16-byte aligned, cols % 8 == 0,
+// asynchronous: complete after stage_wait() and a barrier.
+__device__ __forceinline__ void stage_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
 __device__ __forceinline__ void stage_rows(bf16* dst, int ldd, const bf16* src, int lds, int cols, int valid, int cnt, bool vec) {
   if (vec) {
     const int c8 = (threadIdx.x & 7) * 8;
-    for (int t = threadIdx.x >> 3; t < kGC; t += kGmThreads / 8)
+#pragma unroll
+    for (int tr = 0; tr < kGC; tr += kGmThreads / 8) {
+      const int t = tr + (threadIdx.x >> 3);
       for (int c = c8; c < cols; c += 64) {
-        uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (t < cnt && c < valid) v = *reinterpret_cast<const uint4*>(src + (size_t)t * lds + c);
-        *reinterpret_cast<uint4*>(dst + t * ldd + c) = v;
+        if (t < cnt && c < valid) cp16(dst + t * ldd + c, src + (size_t)t * lds + c);
+        else *reinterpret_cast<uint4*>(dst + t * ldd + c) = make_uint4(0u, 0u, 0u, 0u);
       }
+    }
   } else {
     for (int i = threadIdx.x; i < kGC * cols; i += kGmThreads) {
       const int t = i / cols, c = i - t * cols;
       dst[t * ldd + c] = (t < cnt && c < valid) ? src[(size_t)t * lds + c] : from_f<bf16>(0.f);
     }
   }
+}
+
+// Summed log decays of a chunk, 64 channels from `src` (zero past cnt rows and dn channels), into shared memory.
+__device__ __forceinline__ void stage_decays(float* dst, const float* src, int HD, int dn, int cnt, bool vec) {
+  if (vec) {
+    const int c = (threadIdx.x & 15) * 4;
+#pragma unroll
+    for (int tr = 0; tr < kGC; tr += kGmThreads / 16) {
+      const int t = tr + (threadIdx.x >> 4);
+      if (t < cnt && c < dn) cp16(dst + t * kGbLd + c, src + (size_t)t * HD + c);
+      else *reinterpret_cast<float4*>(dst + t * kGbLd + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  } else {
+    for (int i = threadIdx.x; i < kGC * 64; i += kGmThreads) {
+      const int t = i >> 6, d = i & 63;
+      dst[t * kGbLd + d] = (t < cnt && d < dn) ? src[(size_t)t * HD + d] : 0.f;
+    }
+  }
+}
+
+// Log decay of the chunk's sub-blocks (their last token's sum).
+__device__ __forceinline__ bool sub_block_totals(float* tot, const float* bl, int cnt) {
+  bool deep = false;
+  for (int i = threadIdx.x; i < kGSubs * 64; i += kGmThreads) {
+    const int s = i >> 6, t = min(cnt, (s + 1) * kGS) - 1;
+    const float x = s * kGS < cnt ? bl[t * kGbLd + (i & 63)] : 0.f;
+    tot[i] = x;
+    deep |= x < kSplitLimit;
+  }
+  return deep;
 }
 
 // grid (chunks, H * d tiles, B): 64 channels x vdim of a chunk's contribution.
@@ -328,31 +366,25 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_ke
   const bf16* base = reinterpret_cast<const bf16*>(p.p) + (size_t)(b * p.T + t0) * p.ldp;
   const float* bl = w.bl + (size_t)(b * p.T + t0) * HD + h * p.dim + d0;
   const int dn = min(64, p.dim - d0);
-  for (int i = tid; i < kGSubs * 64; i += kGmThreads) {
-    const int s = i >> 6, d = i & 63, t = min(cnt, (s + 1) * kGS) - 1;
-    sm.tot[i] = (s * kGS < cnt && d < dn) ? bl[(size_t)t * HD + d] : 0.f;
-  }
+  stage_decays(sm.bl, bl, HD, dn, cnt, vec);
+  stage_rows(sm.k, kGmLd, base + p.k_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
   stage_rows(sm.v, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  stage_wait();
   __syncthreads();
-  const bf16* kp = base + p.k_off + h * p.dim + d0;
+  sub_block_totals(sm.tot, sm.bl, cnt);
+  __syncthreads();
 #pragma unroll 4
   for (int i = tid; i < kGC * 32; i += kGmThreads) {      // pairs of channels
     const int t = i >> 5, d = (i & 31) * 2, s = t / kGS;
-    float x = 0.f, y = 0.f;
-    if (t < cnt) {
-      if (d < dn) {
-        float e = sm.tot[s * 64 + d] - bl[(size_t)t * HD + d];
-        for (int m = s + 1; m < kGSubs; ++m) e += sm.tot[m * 64 + d];
-        x = to_f(kp[(size_t)t * p.ldp + d]) * expf(e);
-      }
-      if (d + 1 < dn) {
-        float e = sm.tot[s * 64 + d + 1] - bl[(size_t)t * HD + d + 1];
-        for (int m = s + 1; m < kGSubs; ++m) e += sm.tot[m * 64 + d + 1];
-        y = to_f(kp[(size_t)t * p.ldp + d + 1]) * expf(e);
-      }
-    }
+    const float2 bb = *reinterpret_cast<const float2*>(sm.bl + t * kGbLd + d);
+    const uint32_t kk = *reinterpret_cast<const uint32_t*>(sm.k + t * kGmLd + d);
+    float ex = sm.tot[s * 64 + d] - bb.x, ey = sm.tot[s * 64 + d + 1] - bb.y;
+#pragma unroll
+    for (int m = 1; m < kGSubs; ++m)
+      if (m > s) { ex += sm.tot[m * 64 + d]; ey += sm.tot[m * 64 + d + 1]; }
     uint32_t hi, lo;
-    split_bf16(x, y, hi, lo);
+    split_bf16(bf_lo(kk) * __expf(ex), bf_hi(kk) * __expf(ey), hi, lo);
+    if (t >= cnt) hi = lo = 0u;
     *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
     *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
   }
@@ -398,7 +430,7 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_ke
 template <int VD> struct GlaOutSmem {
   bf16 q[kGC * kGmLd], k[kGC * kGmLd];           // as they are
   bf16 khi[kGC * kGmLd], klo[kGC * kGmLd];       // k decayed to the end of its sub-block
-  float bl[kGC * 68];                            // summed log decays
+  float bl[kGC * kGbLd];                         // summed log decays
   float tot[kGSubs * 64];                        // log decay of a whole sub-block
   float fac[10 * 64];                            // factors of the block pairs and of the chunk's start, see below
   bf16 shi[64 * (VD + 8)], slo[64 * (VD + 8)];   // a tile of the state; at the end v
@@ -437,48 +469,41 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
     __syncthreads();                   // the tile before is no longer read
     stage_rows(sm.q, kGmLd, base + p.q_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
     stage_rows(sm.k, kGmLd, base + p.k_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
-    for (int i = tid; i < kGC * 64; i += kGmThreads) {
-      const int t = i >> 6, d = i & 63;
-      sm.bl[t * 68 + d] = (t < cnt && d < dn) ? blg[(size_t)t * HD + d0 + d] : 0.f;
+    stage_decays(sm.bl, blg + d0, HD, dn, cnt, vec);
+#pragma unroll 8
+    for (int i = tid; i < 64 * (VD / 4); i += kGmThreads) {     // state, four columns at a time (a row is padded to fours)
+      const int d = i / (VD / 4), v = (i - d * (VD / 4)) * 4;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (d < dn && v < p.lds) x = *reinterpret_cast<const float4*>(S + (size_t)(d0 + d) * p.lds + v);
+      uint32_t h0, l0, h1, l1;
+      split_bf16(x.x, x.y, h0, l0);
+      split_bf16(x.z, x.w, h1, l1);
+      *reinterpret_cast<uint2*>(sm.shi + d * (VD + 8) + v) = make_uint2(h0, h1);
+      *reinterpret_cast<uint2*>(sm.slo + d * (VD + 8) + v) = make_uint2(l0, l1);
     }
-    for (int i = tid; i < 64 * (VD / 2); i += kGmThreads) {     // state, in pairs of columns
-      const int d = i / (VD / 2), v = (i - d * (VD / 2)) * 2;
-      float2 x = make_float2(0.f, 0.f);
-      if (d < dn && v < p.lds) x = *reinterpret_cast<const float2*>(S + (size_t)(d0 + d) * p.lds + v);
-      uint32_t hi, lo;
-      split_bf16(x.x, x.y, hi, lo);
-      *reinterpret_cast<uint32_t*>(sm.shi + d * (VD + 8) + v) = hi;
-      *reinterpret_cast<uint32_t*>(sm.slo + d * (VD + 8) + v) = lo;
-    }
+    stage_wait();
     __syncthreads();
-    bool deep = false;                 // some channel of the tile decays past the limit inside a sub-block
-    for (int i = tid; i < kGSubs * 64; i += kGmThreads) {
-      const int s = i >> 6, t = min(cnt, (s + 1) * kGS) - 1;
-      const float x = s * kGS < cnt ? sm.bl[t * 68 + (i & 63)] : 0.f;
-      sm.tot[i] = x;
-      deep |= x < kSplitLimit;
-    }
-    deep = __syncthreads_or(deep);
+    const bool deep = __syncthreads_or(sub_block_totals(sm.tot, sm.bl, cnt));   // some channel decays past the limit in a sub-block
     if (tid < 64) {
       const float a0 = sm.tot[tid], a1 = sm.tot[64 + tid], a2 = sm.tot[128 + tid], a3 = sm.tot[192 + tid];
       float* f = sm.fac + tid;
-      f[0 * 64] = expf(a1);            // between sub-blocks 2 and 0
-      f[1 * 64] = expf(a2);            // 3 and 1
-      f[2 * 64] = expf(a1 + a2);       // 3 and 0
-      f[3 * 64] = expf(a0);            // from the chunk's start to sub-block 1, 2, 3
-      f[4 * 64] = expf(a0 + a1);
-      f[5 * 64] = expf(a0 + a1 + a2);
-      f[6 * 64] = deep ? 0.f : expf(-a0);      // inside sub-block 0 .. 3
-      f[7 * 64] = deep ? 0.f : expf(-a1);
-      f[8 * 64] = deep ? 0.f : expf(-a2);
-      f[9 * 64] = deep ? 0.f : expf(-a3);
+      f[0 * 64] = __expf(a1);            // between sub-blocks 2 and 0
+      f[1 * 64] = __expf(a2);            // 3 and 1
+      f[2 * 64] = __expf(a1 + a2);       // 3 and 0
+      f[3 * 64] = __expf(a0);            // from the chunk's start to sub-block 1, 2, 3
+      f[4 * 64] = __expf(a0 + a1);
+      f[5 * 64] = __expf(a0 + a1 + a2);
+      f[6 * 64] = deep ? 0.f : __expf(-a0);      // inside sub-block 0 .. 3
+      f[7 * 64] = deep ? 0.f : __expf(-a1);
+      f[8 * 64] = deep ? 0.f : __expf(-a2);
+      f[9 * 64] = deep ? 0.f : __expf(-a3);
     }
     for (int i = tid; i < kGC * 32; i += kGmThreads) {
       const int t = i >> 5, d = (i & 31) * 2;
       const uint32_t kk = *reinterpret_cast<const uint32_t*>(sm.k + t * kGmLd + d);
       const float* tt = sm.tot + (t / kGS) * 64 + d;
       uint32_t hi, lo;
-      split_bf16(bf_lo(kk) * expf(tt[0] - sm.bl[t * 68 + d]), bf_hi(kk) * expf(tt[1] - sm.bl[t * 68 + d + 1]), hi, lo);
+      split_bf16(bf_lo(kk) * __expf(tt[0] - sm.bl[t * kGbLd + d]), bf_hi(kk) * __expf(tt[1] - sm.bl[t * kGbLd + d + 1]), hi, lo);
       if (t >= cnt) hi = lo = 0u;
       *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
       *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
@@ -493,8 +518,8 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
       for (int j = 0; j < 4; ++j) {
         const int r = (j & 1) ? rb : ra, c = kk + c2 + (j >> 1) * 8;
         const uint32_t qq = *reinterpret_cast<const uint32_t*>(sm.q + r * kGmLd + c);
-        qd[j][0] = bf_lo(qq) * qscale * expf(sm.bl[r * 68 + c]);
-        qd[j][1] = bf_hi(qq) * qscale * expf(sm.bl[r * 68 + c + 1]);
+        qd[j][0] = bf_lo(qq) * qscale * __expf(sm.bl[r * kGbLd + c]);
+        qd[j][1] = bf_hi(qq) * qscale * __expf(sm.bl[r * kGbLd + c + 1]);
       }
       auto fragment = [&](const float* f, uint32_t (&hi)[4], uint32_t (&lo)[4]) {   // f: per-channel factor or null
 #pragma unroll
@@ -517,26 +542,32 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
         const int off = (j * 16 + (lane & 7) + ((lane >> 4) << 3)) * kGmLd + kk + ((lane >> 3) & 1) * 8;
         ldsm_x4(kh, sm.khi + off);
         ldsm_x4(kl, sm.klo + off);
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          mma_bf16(sc[j][x], hi, kh[2 * x], kh[2 * x + 1]);
-          mma_bf16(sc[j][x], hi, kl[2 * x], kl[2 * x + 1]);
-          mma_bf16(sc[j][x], lo, kh[2 * x], kh[2 * x + 1]);
-        }
+        mma_bf16(sc[j][0], hi, kh[0], kh[1]);
+        mma_bf16(sc[j][1], hi, kh[2], kh[3]);
+        mma_bf16(sc[j][0], hi, kl[0], kl[1]);
+        mma_bf16(sc[j][1], hi, kl[2], kl[3]);
+        mma_bf16(sc[j][0], lo, kh[0], kh[1]);
+        mma_bf16(sc[j][1], lo, kh[2], kh[3]);
       }
       fragment(warp == 0 ? nullptr : sm.fac + (2 + warp) * 64, hi, lo);
 #pragma unroll
-      for (int v = 0; v < VD / 16; ++v) {
-        uint32_t sh[4], sl[4];
-        const int off = (kk + (lane & 15)) * (VD + 8) + v * 16 + (lane >> 4) * 8;
-        ldsm_x4_t(sh, sm.shi + off);
-        ldsm_x4_t(sl, sm.slo + off);
+      for (int v = 0; v < VD / 16; v += 2) {         // eight independent products before an accumulator comes again
+        uint32_t sh[2][4], sl[2][4];
 #pragma unroll
-        for (int x = 0; x < 2; ++x) {
-          mma_bf16(o[2 * v + x], hi, sh[2 * x], sh[2 * x + 1]);
-          mma_bf16(o[2 * v + x], hi, sl[2 * x], sl[2 * x + 1]);
-          mma_bf16(o[2 * v + x], lo, sh[2 * x], sh[2 * x + 1]);
+        for (int y = 0; y < 2; ++y) {
+          const int off = (kk + (lane & 15)) * (VD + 8) + (v + y) * 16 + (lane >> 4) * 8;
+          ldsm_x4_t(sh[y], sm.shi + off);
+          ldsm_x4_t(sl[y], sm.slo + off);
         }
+#pragma unroll
+        for (int term = 0; term < 3; ++term)
+#pragma unroll
+          for (int y = 0; y < 2; ++y)
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+              const uint32_t(&bb)[4] = term == 1 ? sl[y] : sh[y];
+              mma_bf16(o[2 * (v + y) + x], term == 2 ? lo : hi, bb[2 * x], bb[2 * x + 1]);
+            }
       }
     }
     if (deep) {                        // the pairs of this warp's own sub-block, one exponential each
@@ -551,7 +582,7 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
             if (s > t || t >= cnt) continue;
             float sum = 0.f;
             for (int d = 0; d < dn; ++d)
-              sum += to_f(sm.q[t * kGmLd + d]) * expf(sm.bl[t * 68 + d] - sm.bl[s * 68 + d]) * to_f(sm.k[s * kGmLd + d]);
+              sum += to_f(sm.q[t * kGmLd + d]) * __expf(sm.bl[t * kGbLd + d] - sm.bl[s * kGbLd + d]) * to_f(sm.k[s * kGmLd + d]);
             sc[j][x][e] += sum * qscale;
           }
       }
@@ -559,6 +590,7 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
   }
   __syncthreads();
   stage_rows(sm.shi, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  stage_wait();
   __syncthreads();
 #pragma unroll
   for (int j = 0; j < kGSubs; ++j) {

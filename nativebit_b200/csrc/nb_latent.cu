@@ -54,6 +54,21 @@ template <typename T> __global__ void __launch_bounds__(kPrepThreads) latent_pre
   }
 }
 
+// Eight bf16 values (four pairs) of a rotated vector; c, s: their entries of the tables.
+__device__ __forceinline__ uint4 rotate8(uint4 t, const float* __restrict__ c, const float* __restrict__ s) {
+  const float4 c0 = __ldg(reinterpret_cast<const float4*>(c)), c1 = __ldg(reinterpret_cast<const float4*>(c + 4));
+  const float4 s0 = __ldg(reinterpret_cast<const float4*>(s)), s1 = __ldg(reinterpret_cast<const float4*>(s + 4));
+  const float cs[8] = {c0.x, c0.y, c0.z, c0.w, c1.x, c1.y, c1.z, c1.w}, sn[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
+  const uint32_t u[4] = {t.x, t.y, t.z, t.w};
+  uint32_t r[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float x = bf_lo(u[e]), y = bf_hi(u[e]);
+    r[e] = pack_bf16(x * cs[2 * e] - y * sn[2 * e], y * cs[2 * e + 1] + x * sn[2 * e + 1]);
+  }
+  return make_uint4(r[0], r[1], r[2], r[3]);
+}
+
 // The same for bf16 rows whose pieces are all multiples of eight: one warp per query latent, one per key/value row, sixteen
 // bytes per lane and load, everything of a row in flight at once and kept in registers between the norm's two passes.
 constexpr int kPvQ = 8;                // loads per lane: up to 2048 columns
@@ -107,19 +122,9 @@ __global__ void __launch_bounds__(256) latent_prepare_vec_kernel(const nb_latent
   const bf16* kv = a + p.kv_off;
   if (p.rank <= 512) norm_row_bf16<2>(kv, p.kv_norm, p.eps, p.rank, c, lane);
   else norm_row_bf16<kPvQ>(kv, p.kv_norm, p.eps, p.rank, c, lane);
-  for (int d = lane * 8; d < p.rot; d += 256) {
-    const uint4 t = *reinterpret_cast<const uint4*>(kv + p.rank + d);
-    const uint32_t u[4] = {t.x, t.y, t.z, t.w};
-    uint32_t r[4];
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float2 cs = *reinterpret_cast<const float2*>(p.cos2 + (size_t)pos * p.rot + d + 2 * e);
-      const float2 sn = *reinterpret_cast<const float2*>(p.sin2 + (size_t)pos * p.rot + d + 2 * e);
-      const float x = bf_lo(u[e]), y = bf_hi(u[e]);
-      r[e] = pack_bf16(x * cs.x - y * sn.x, y * cs.y + x * sn.y);
-    }
-    *reinterpret_cast<uint4*>(c + p.rank + d) = make_uint4(r[0], r[1], r[2], r[3]);
-  }
+  const float *cs = p.cos2 + (size_t)pos * p.rot, *sn = p.sin2 + (size_t)pos * p.rot;
+  for (int d = lane * 8; d < p.rot; d += 256)
+    *reinterpret_cast<uint4*>(c + p.rank + d) = rotate8(*reinterpret_cast<const uint4*>(kv + p.rank + d), cs + d, sn + d);
 }
 
 // ---- a portion of a prompt, fp32.  A CTA owns 16 queries of one head and walks the visible keys in chunks of 32 staged
@@ -228,7 +233,7 @@ __global__ void __launch_bounds__(kLThreads) latent_attention_f32_kernel(const n
 constexpr int kTQ = 64, kTK = 64, kTThreads = 128;
 
 template <int VD>
-__global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const nb_latent_attention_args p, int dk16, int vec) {
+__global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const nb_latent_attention_args p, int dk16, int vec, int qvec) {
   extern __shared__ __align__(16) bf16 tsm[];
   const int dk = p.dim + p.rot, dkp = dk16 + 8;
   constexpr int vp = VD + 8;
@@ -291,18 +296,39 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  copy_tile(0, 0);
-  for (int i = tid; i < kTQ * dk; i += kTThreads) {
-    const int r = i / dk, d = i - r * dk, t = min(q0 + r, p.T - 1);
-    const bf16* qr = q + (size_t)(b * p.T + t) * p.ldq + h * dk;
-    bf16 v;
-    if (d < p.dim) {
-      v = qr[d];
-    } else {
-      const size_t at = (size_t)(p.pos0 + t) * p.rot;
-      v = from_f<bf16>(rotated([&](int j) { return to_f(qr[p.dim + j]); }, p.cos2 + at, p.sin2 + at, d - p.dim));
+  if (qvec) {                                   // travels with the first tile; the rotated part through registers
+    const int c8 = (tid & 7) * 8;
+#pragma unroll
+    for (int r0 = 0; r0 < kTQ; r0 += kTThreads / 8) {
+      const int r = r0 + (tid >> 3), t = min(q0 + r, p.T - 1);
+      const bf16* qr = q + (size_t)(b * p.T + t) * p.ldq + h * dk;
+      for (int c = c8; c < p.dim; c += 64) cp16(q_s + r * dkp + c, qr + c);
     }
-    q_s[r * dkp + d] = v;
+  }
+  copy_tile(0, 0);
+  if (qvec) {
+    const int c8 = (tid & 7) * 8;
+#pragma unroll
+    for (int r0 = 0; r0 < kTQ; r0 += kTThreads / 8) {
+      const int r = r0 + (tid >> 3), t = min(q0 + r, p.T - 1);
+      const bf16* qr = q + (size_t)(b * p.T + t) * p.ldq + h * dk + p.dim;
+      const float *cs = p.cos2 + (size_t)(p.pos0 + t) * p.rot, *sn = p.sin2 + (size_t)(p.pos0 + t) * p.rot;
+      for (int c = c8; c < p.rot; c += 64)
+        *reinterpret_cast<uint4*>(q_s + r * dkp + p.dim + c) = rotate8(*reinterpret_cast<const uint4*>(qr + c), cs + c, sn + c);
+    }
+  } else {
+    for (int i = tid; i < kTQ * dk; i += kTThreads) {
+      const int r = i / dk, d = i - r * dk, t = min(q0 + r, p.T - 1);
+      const bf16* qr = q + (size_t)(b * p.T + t) * p.ldq + h * dk;
+      bf16 v;
+      if (d < p.dim) {
+        v = qr[d];
+      } else {
+        const size_t at = (size_t)(p.pos0 + t) * p.rot;
+        v = from_f<bf16>(rotated([&](int j) { return to_f(qr[p.dim + j]); }, p.cos2 + at, p.sin2 + at, d - p.dim));
+      }
+      q_s[r * dkp + d] = v;
+    }
   }
 
   // this lane's two rows of the warp's 16 queries: lane / 4 and lane / 4 + 8
@@ -390,13 +416,16 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
         split_bf16(x, y, hi[j], lo[j]);
       }
 #pragma unroll
-      for (int n = 0; n < VD / 16; ++n) {
-        uint32_t bb[4];
-        ldsm_x4_t(bb, vt + (kk * 16 + (lane & 15)) * vp + n * 16 + (lane >> 4) * 8);
-        mma_bf16(o[2 * n], hi, bb[0], bb[1]);
-        mma_bf16(o[2 * n + 1], hi, bb[2], bb[3]);
-        mma_bf16(o[2 * n], lo, bb[0], bb[1]);
-        mma_bf16(o[2 * n + 1], lo, bb[2], bb[3]);
+      for (int n = 0; n < VD / 16; n += 2) {           // four independent products before an accumulator comes again
+        uint32_t bb[2][4];
+        ldsm_x4_t(bb[0], vt + (kk * 16 + (lane & 15)) * vp + n * 16 + (lane >> 4) * 8);
+        ldsm_x4_t(bb[1], vt + (kk * 16 + (lane & 15)) * vp + n * 16 + 16 + (lane >> 4) * 8);
+#pragma unroll
+        for (int term = 0; term < 2; ++term)
+#pragma unroll
+          for (int y = 0; y < 2; ++y)
+#pragma unroll
+            for (int x = 0; x < 2; ++x) mma_bf16(o[2 * (n + y) + x], term ? lo : hi, bb[y][2 * x], bb[y][2 * x + 1]);
       }
     }
     __syncthreads();                                   // before the stage is filled again
@@ -459,19 +488,22 @@ __device__ __forceinline__ float2 pair_at(const float* r) { return *reinterpret_
 template <typename T> __host__ __device__ inline int staged_row(int rdp) { return rdp % (32 / (int)sizeof(T)) ? rdp : rdp + 16 / (int)sizeof(T); }
 
 template <typename T>
-__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_latent_decode_args p, int stage) {
+__global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_latent_decode_args p, int stage) {
   extern __shared__ __align__(16) float dsm[];
-  __shared__ float red[2 * kLdWarps], red2[kLdWarps], red3[kLdWarps];
+  __shared__ float red[kLdWarps], red2[kLdWarps], red3[kLdWarps];
   cg::cluster_group cluster = cg::this_cluster();
   const int S = (int)cluster.num_blocks(), rank_id = (int)cluster.block_rank();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int rd = p.rank + p.rot, dk = p.dim + p.rot, rdp = (rd + 7) & ~7, ldr = staged_row<T>(rdp);
   float* qa = dsm;                     // [rdp] q' and the rotated query part: what the cached rows are multiplied with
   float* ol = qa + rdp;                // [rdp] merged latent
-  float* xch = ol + rdp;               // [rdp + 8] what the other CTAs read: weighted latent, maximum, sum
-  float* qn = xch + rdp + 8;           // [dk] this head's query
-  float* part = qn + ((dk + 7) & ~7);  // [kLdThreads * 2] partial sums
-  float* sc = part + 2 * kLdThreads;   // [stage] scores, then weights, of the staged keys
+  float* qn = ol + rdp;                // [dk] this head's query
+  float* cs = qn + ((dk + 7) & ~7);    // [rot] the position's rotary entries
+  float* sn = cs + ((p.rot + 7) & ~7);
+  float* part = sn + ((p.rot + 7) & ~7);   // [kLdThreads * 2] partial sums
+  const int pairs = (p.rank + 1) / 2, pper = (pairs + S - 1) / S, slot = (2 * pper + 2 + 3) & ~3;
+  float* xch = part + 2 * kLdThreads;  // [S][slot] what the CTAs send: their part of this CTA's slice, maximum, sum
+  float* sc = xch + S * slot;          // [stage] scores, then weights, of the staged keys
   T* rows = reinterpret_cast<T*>(sc + ((stage + 3) & ~3));   // [stage][ldr]
 
   // The position was written at the end of the step before, the rows below it in earlier steps or the prompt.
@@ -494,7 +526,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
   request(0, min(stage, cnt));
 
   // W_uk: this CTA's slice of columns (pairs), the d range split over groups of threads
-  const int pairs = (p.rank + 1) / 2, pper = (pairs + S - 1) / S, p0 = rank_id * pper, pn = max(0, min(pairs, p0 + pper) - p0);
+  const int p0 = rank_id * pper, pn = max(0, min(pairs, p0 + pper) - p0);
   const bf16* uk = reinterpret_cast<const bf16*>(p.uk) + (size_t)h * p.dim * p.ldu;
   const int cols0 = min(pn, kLdThreads), groups0 = cols0 ? kLdThreads / cols0 : 1, g0 = cols0 ? tid / cols0 : 0, c0 = cols0 ? tid - g0 * cols0 : 0;
   const bool pre = pn > 0 && pn <= kLdThreads && (p.dim + groups0 - 1) / groups0 <= kLdPre;
@@ -510,35 +542,60 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
     const int v = i / ((p.rank + 63) / 64), c = i - v * ((p.rank + 63) / 64);
     prefetch_l2(uv + (size_t)(v0 + v) * p.ldu + c * 64);
   }
-  const float *cs = p.cos2 + (size_t)pos * p.rot, *sn = p.sin2 + (size_t)pos * p.rot;
+  // the position's rotary entries and the norm's weights
+  for (int i = tid; i < p.rot; i += kLdThreads) { cs[i] = p.cos2[(size_t)pos * p.rot + i]; sn[i] = p.sin2[(size_t)pos * p.rot + i]; }
+  const int mine = (int)pos - k0;      // this position's place among this CTA's keys, if 0 <= mine < cnt
+  const bool holds = mine >= 0 && mine < cnt;
+  constexpr int kKv = 2 * kLdCols;     // elements of the position's latent per thread
+  float kvw[kKv], kvv[kKv];
+  if (p.kv_off >= 0 && holds) {
+#pragma unroll
+    for (int u = 0; u < kKv; ++u) kvw[u] = tid + u * kLdThreads < p.rank ? p.kv_norm[tid + u * kLdThreads] : 0.f;
+  }
+  cluster.barrier_arrive();
 
   pdl_enter();
   for (int i = tid; i < dk; i += kLdThreads) qn[i] = p.q[(size_t)b * p.ldq + h * dk + i];
+  const float gate = p.a[(size_t)b * p.lda + p.g_off + h];
   for (int i = rd + tid; i < rdp; i += kLdThreads) qa[i] = 0.f;
-  // this position's row: from the projection (and written to the cache by one CTA) or from the cache
-  const int mine = (int)pos - k0;      // its place among this CTA's keys, if 0 <= mine < cnt
-  const bool holds = mine >= 0 && mine < cnt;
-  float mean, inv = 0.f;
+  // this position's row, into its staged place: from the projection (and then written to the cache by one CTA) or from
+  // the cache.  With more keys than are staged at a time it waits in its registers for its turn.
+  float inv = 0.f;
   const float* kv = p.a + (size_t)b * p.lda + max(p.kv_off, 0);
-  if (p.kv_off >= 0 && holds)          // block-uniform
-    norm_stats<kLdWarps>(NB_NORM_RMS, p.rank, p.eps, red,
-                         [&](auto f) { for (int i = tid; i < p.rank; i += kLdThreads) f(kv[i]); }, mean, inv);
+  if (p.kv_off >= 0 && holds) {        // block-uniform
+    float ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < kKv; ++u) {
+      kvv[u] = tid + u * kLdThreads < p.rank ? kv[tid + u * kLdThreads] : 0.f;
+      ss += kvv[u] * kvv[u];
+    }
+    inv = 1.0f / sqrtf(block_sum<kLdWarps>(ss, red) / (float)p.rank + p.eps);
+  } else {
+    __syncthreads();                   // the query and the rotary entries
+  }
   auto put_row = [&](T* dst) {         // dst: the staged row
     T* crow = cache + (size_t)pos * p.ldc;
-    for (int i = tid; i < rdp; i += kLdThreads) {
-      T v = from_f<T>(0.f);
-      if (i < rd) {
-        if (p.kv_off >= 0) {
-          v = from_f<T>(i < p.rank ? kv[i] * inv * p.kv_norm[i] : rotated([&](int j) { return kv[p.rank + j]; }, cs, sn, i - p.rank));
+    if (p.kv_off >= 0) {
+#pragma unroll
+      for (int u = 0; u < kKv; ++u) {
+        const int i = tid + u * kLdThreads;
+        if (i < p.rank) {
+          const T v = from_f<T>(kvv[u] * inv * kvw[u]);
+          dst[i] = v;
           if (h == 0) crow[i] = v;
-        } else {
-          v = crow[i];
         }
       }
-      dst[i] = v;
+      for (int d = tid; d < p.rot; d += kLdThreads) {
+        const T v = from_f<T>(rotated([&](int j) { return kv[p.rank + j]; }, cs, sn, d));
+        dst[p.rank + d] = v;
+        if (h == 0) crow[p.rank + d] = v;
+      }
+    } else {
+      for (int i = tid; i < rd; i += kLdThreads) dst[i] = crow[i];
     }
+    for (int i = rd + tid; i < rdp; i += kLdThreads) dst[i] = from_f<T>(0.f);
   };
-  cluster.sync();                      // every CTA of the cluster runs: its shared memory may be written from here on
+  if (mine >= 0 && mine < min(stage, cnt)) put_row(rows + (size_t)mine * ldr);
   for (int d = tid; d < p.rot; d += kLdThreads) qa[p.rank + d] = rotated([&](int j) { return qn[p.dim + j]; }, cs, sn, d);
 
   // q'[j] = sum_d W_uk[h][d][j] q[d]
@@ -561,6 +618,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
       }
     }
     part[2 * tid] = x; part[2 * tid + 1] = y;
+    if (base == 0) cluster.barrier_wait();     // every CTA of the cluster runs: its shared memory may be written from here on
     __syncthreads();
     for (int i = tid; i < 2 * cols; i += kLdThreads) {
       float v = 0.f;
@@ -571,6 +629,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
     }
     __syncthreads();
   }
+  if (pn == 0) cluster.barrier_wait();
   cluster.sync();
 
   // softmax and weighted latent over the staged rows.  Scores: four lanes share a key, sixteen bytes at a time.  Latent: a
@@ -586,7 +645,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
       __syncthreads();                 // the rows and weights before are no longer read
       request(base, nk);
     }
-    if (mine >= base && mine < base + nk) put_row(rows + (size_t)(mine - base) * ldr);
+    if (base > 0 && mine >= base && mine < base + nk) put_row(rows + (size_t)(mine - base) * ldr);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     float mx = -FLT_MAX;
@@ -635,6 +694,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
       }
     }
   }
+  // every CTA sends the parts of its weighted latent to the CTAs that merge them: slice r (2 * pper columns) to CTA r
 #pragma unroll
   for (int u = 0; u < kLdCols; ++u) {
     if (u * kLdThreads < pairs) {      // block-uniform
@@ -644,48 +704,80 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const nb_late
       for (int i = tid; i < 2 * cols; i += kLdThreads) {
         float v = 0.f;
         for (int g = 0; g < groups; ++g) v += part[2 * g * wcols + i];
-        xch[2 * u * kLdThreads + i] = v;
+        const int col = 2 * u * kLdThreads + i, to = col / (2 * pper);
+        cluster.map_shared_rank(xch, to)[rank_id * slot + col - to * 2 * pper] = v;
       }
       __syncthreads();
     }
   }
-  if (tid == 0) { xch[rdp] = m; xch[rdp + 1] = l; }
+  if (tid < S) {
+    float* x = cluster.map_shared_rank(xch, tid) + rank_id * slot + 2 * pper;
+    x[0] = m;
+    x[1] = l;
+  }
+  // rows of W_uv for the last product, two per warp, requested ahead of the exchange
+  constexpr int kUvPre = 4;
+  const bool upre = p.rank <= 512 && v1 - v0 <= 2 * kLdWarps;
+  uint4 uvr[kUvPre];
+#pragma unroll
+  for (int i = 0; i < kUvPre; ++i) {
+    const int v = v0 + warp + (i >> 1) * kLdWarps, c = (i & 1) * 256 + lane * 8;
+    uvr[i] = (upre && v < v1 && c < p.rank) ? __ldg(reinterpret_cast<const uint4*>(uv + (size_t)v * p.ldu + c)) : make_uint4(0u, 0u, 0u, 0u);
+  }
   cluster.sync();
   // this CTA's slice of the merged latent, to everyone
   {
     float m_all = -FLT_MAX, den = 0.f, wr[8];
-    for (int r = 0; r < S; ++r) m_all = fmaxf(m_all, cluster.map_shared_rank(xch, r)[rdp]);
+#pragma unroll
+    for (int r = 0; r < 8; ++r)
+      if (r < S) m_all = fmaxf(m_all, xch[r * slot + 2 * pper]);
 #pragma unroll
     for (int r = 0; r < 8; ++r) {      // a CTA without keys has maximum -FLT_MAX and sum 0
       wr[r] = 0.f;
       if (r < S) {
-        const float* rx = cluster.map_shared_rank(xch, r);
-        wr[r] = expf(rx[rdp] - m_all);
-        den += wr[r] * rx[rdp + 1];
+        wr[r] = expf(xch[r * slot + 2 * pper] - m_all);
+        den += wr[r] * xch[r * slot + 2 * pper + 1];
       }
     }
-    for (int i = 2 * p0 + tid; i < min(p.rank, 2 * (p0 + pn)); i += kLdThreads) {
+    for (int i = tid; i < min(2 * pn, p.rank - 2 * p0); i += kLdThreads) {
       float num = 0.f;
 #pragma unroll
       for (int r = 0; r < 8; ++r)
-        if (r < S) num += wr[r] * cluster.map_shared_rank(xch, r)[i];
+        if (r < S) num += wr[r] * xch[r * slot + i];
       const float v = num / den;
-      for (int r = 0; r < S; ++r) cluster.map_shared_rank(ol, r)[i] = v;
+      for (int r = 0; r < S; ++r) cluster.map_shared_rank(ol, r)[2 * p0 + i] = v;
     }
   }
   for (int i = p.rank + tid; i < ((p.rank + 7) & ~7); i += kLdThreads) ol[i] = 0.f;   // W_uv is read in eights
   cluster.sync();                      // also: nobody reads another CTA's shared memory after this
-  const float g = sigmoid_f(p.a[(size_t)b * p.lda + p.g_off + h]);
-  for (int v = v0 + warp; v < v1; v += kLdWarps) {
-    const bf16* wv = uv + (size_t)v * p.ldu;
-    float s = 0.f;
-    for (int i = lane * 8; i < p.rank; i += 256) s += dot16<bf16>(wv + i, ol + i);
-    s = warp_sum(s);
-    if (lane == 0) p.out[(size_t)b * p.ldo + h * p.vdim + v] = s * g;
+  const float g = sigmoid_f(gate);
+  if (upre) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int v = v0 + warp + r * kLdWarps;
+      if (v < v1) {
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int c = i * 256 + lane * 8;
+          if (c < p.rank) s += dot16<bf16>(&uvr[2 * r + i], ol + c);
+        }
+        s = warp_sum(s);
+        if (lane == 0) p.out[(size_t)b * p.ldo + h * p.vdim + v] = s * g;
+      }
+    }
+  } else {
+    for (int v = v0 + warp; v < v1; v += kLdWarps) {
+      const bf16* wv = uv + (size_t)v * p.ldu;
+      float s = 0.f;
+      for (int i = lane * 8; i < p.rank; i += 256) s += dot16<bf16>(wv + i, ol + i);
+      s = warp_sum(s);
+      if (lane == 0) p.out[(size_t)b * p.ldo + h * p.vdim + v] = s * g;
+    }
   }
 }
 
-constexpr size_t kLatentMaxSmem = 200 * 1024;
+constexpr size_t kLatentMaxSmem = 200 * 1024, kLatentHalfSmem = 110 * 1024;
 
 template <int VPT> static int launch_latent_f32(const nb_latent_attention_args& a, cudaStream_t st) {
   const int dk = a.dim + a.rot;
@@ -718,7 +810,9 @@ template <int VD> static int launch_latent_bf16(const nb_latent_attention_args& 
   // 16-byte copies need every piece of a row to start and end on 16 bytes
   const int vec = a.dim % 8 == 0 && a.rot % 8 == 0 && a.vdim % 8 == 0 && a.rank % 8 == 0 && a.ldkv % 8 == 0 && a.ldc % 8 == 0 &&
                   a.v_off % 8 == 0 && a.ldo % 2 == 0 && (uintptr_t)a.kv % 16 == 0 && (uintptr_t)a.cache % 16 == 0 && (uintptr_t)a.out % 4 == 0;
-  latent_attention_bf16_kernel<VD><<<dim3((a.T + kTQ - 1) / kTQ, a.H, a.B), kTThreads, smem, st>>>(a, dk16, vec);
+  const int qvec = a.dim % 8 == 0 && a.rot % 8 == 0 && a.ldq % 8 == 0 && (uintptr_t)a.q % 16 == 0 && (uintptr_t)a.cos2 % 16 == 0 &&
+                   (uintptr_t)a.sin2 % 16 == 0;
+  latent_attention_bf16_kernel<VD><<<dim3((a.T + kTQ - 1) / kTQ, a.H, a.B), kTThreads, smem, st>>>(a, dk16, vec, qvec);
   return check_launch();
 }
 
@@ -740,8 +834,8 @@ extern "C" int nb_latent_prepare(const nb_latent_prepare_args* a, void* stream) 
   const bool vec = a->dtype == NB_BF16 && a->q_rank % 8 == 0 && a->q_off % 8 == 0 && a->lda % 8 == 0 && a->ldcq % 8 == 0 &&
                    a->q_rank <= 256 * kPvQ && (uintptr_t)a->a % 16 == 0 && (uintptr_t)a->cq % 16 == 0 && (uintptr_t)a->q_norm % 16 == 0 &&
                    (!kv || (a->kv_off % 8 == 0 && a->rank % 8 == 0 && a->rot % 8 == 0 && a->rank <= 256 * kPvQ && a->ldc % 8 == 0 &&
-                            (uintptr_t)a->cache % 16 == 0 && (uintptr_t)a->kv_norm % 16 == 0 && (uintptr_t)a->cos2 % 8 == 0 &&
-                            (uintptr_t)a->sin2 % 8 == 0));
+                            (uintptr_t)a->cache % 16 == 0 && (uintptr_t)a->kv_norm % 16 == 0 && (uintptr_t)a->cos2 % 16 == 0 &&
+                            (uintptr_t)a->sin2 % 16 == 0));
   if (vec) {
     const int rows = a->B * a->T;
     return launch_pdl(latent_prepare_vec_kernel, dim3(((kv ? 2 : 1) * rows + 7) / 8), dim3(256), 0, (cudaStream_t)stream, *a, rows);
@@ -787,10 +881,12 @@ extern "C" int nb_latent_decode(const nb_latent_decode_args* a, void* stream) {
   const int wide = a->cache_dtype == NB_F32;
   const int rdp = (a->rank + a->rot + 7) & ~7;
   const size_t row = (size_t)(wide ? staged_row<float>(rdp) * 4 : staged_row<bf16>(rdp) * 2);
-  const size_t fixed = ((size_t)3 * rdp + 8 + ((a->dim + a->rot + 7) & ~7) + 2 * kLdThreads + 4) * 4;
+  const int pper = ((a->rank + 1) / 2 + S - 1) / S, slot = (2 * pper + 2 + 3) & ~3;
+  const size_t fixed = ((size_t)2 * rdp + ((a->dim + a->rot + 7) & ~7) + 2 * ((a->rot + 7) & ~7) + 2 * kLdThreads + S * slot + 4) * 4;
   if (fixed + 8 * (row + 4) > kLatentMaxSmem) return NB_ERR_SHAPE;
-  // as many of a CTA's rows at a time as shared memory holds
-  const int stage = (int)std::min<size_t>((most + S - 1) / S, (kLatentMaxSmem - fixed) / (row + 4));
+  // as many of a CTA's rows at a time as shared memory holds; two CTAs per SM when they do not all fit one each
+  const size_t budget = (size_t)a->B * a->H * S > 112 && fixed + 8 * (row + 4) <= kLatentHalfSmem ? kLatentHalfSmem : kLatentMaxSmem;
+  const int stage = (int)std::min<size_t>((most + S - 1) / S, (budget - fixed) / (row + 4));
   const size_t smem = fixed + (size_t)((stage + 3) & ~3) * 4 + stage * row;
   static bool done[2][64] = {};
   int dev = 0;

@@ -188,9 +188,9 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 // bytes, 16 per lane), is dealt to the CTA's warps in equal contiguous runs, so every SM and every warp streams the
 // same number of bytes whatever N and K are.  A row that lies in one run is finished by its warp; the parts of a row
 // that runs share are added in warp order after a barrier: no atomics, bit-identical from run to run.  Each warp keeps
-// 8 - 16 items in flight in registers and requests the first ones before the dependency wait; a CTA is small enough
-// that the next launch's CTA fits beside it and starts its own requests while this one drains.
-constexpr int kMvWarps = 8, kMvThreads = kMvWarps * 32, kMvBatch = 8;
+// 8 - 16 items in flight in registers and requests the first ones before the dependency wait.  (Eight warps per CTA, so that the next
+// launch's CTA fits beside it, measured slower: too few bytes in flight.)
+constexpr int kMvWarps = 16, kMvThreads = kMvWarps * 32, kMvBatch = 8;
 
 struct MatvecParams {
   const uint4* w;
@@ -207,8 +207,8 @@ __device__ __forceinline__ uint4 ld_stream(const uint4* p) {
   return v;
 }
 
-template <int NV>   // float4 of the row per thread in the prologue (K <= 1024 * NV, a multiple of 4), 0: any K
-__global__ void __launch_bounds__(kMvThreads, 2) matvec_kernel(const MatvecParams p) {
+template <int NV>   // float4 of the row per thread in the prologue (K <= 2048 * NV, a multiple of 4), 0: any K
+__global__ void __launch_bounds__(kMvThreads, 1) matvec_kernel(const MatvecParams p) {
   extern __shared__ __align__(16) float mv_smem[];
   __shared__ float red[4 * kMvWarps], part_v[2 * kMvWarps];
   __shared__ int part_r[2 * kMvWarps];
@@ -427,9 +427,8 @@ extern "C" int nb_matvec_bf16(const nb_matvec_args* a, void* stream) {
   const cudaStream_t st = (cudaStream_t)stream;
   const bool vec = a->K % 4 == 0 && (uintptr_t)a->x % 16 == 0 && (uintptr_t)a->delta % 16 == 0 && (uintptr_t)a->delta_w % 16 == 0 &&
                    (uintptr_t)a->norm_w % 16 == 0 && (uintptr_t)a->x_out % 16 == 0;
-  if (vec && a->K <= 1024) return launch_matvec<1>(p, G, smem, st);
-  if (vec && a->K <= 2048) return launch_matvec<2>(p, G, smem, st);
-  if (vec && a->K <= 3072) return launch_matvec<3>(p, G, smem, st);
-  if (vec && a->K <= 4096) return launch_matvec<4>(p, G, smem, st);
+  if (vec && a->K <= 2048) return launch_matvec<1>(p, G, smem, st);
+  if (vec && a->K <= 4096) return launch_matvec<2>(p, G, smem, st);
+  if (vec && a->K <= 8192) return launch_matvec<4>(p, G, smem, st);
   return launch_matvec<0>(p, G, smem, st);
 }

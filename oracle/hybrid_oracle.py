@@ -77,27 +77,36 @@ def windowed_attention(q, k, v, scale, window):
     return out
 
 
-def latent_attention(h, w, p, mix, eps, shared=None):
+def exact(x):
+    return x
+
+
+def linear(x, weight, cast=exact):
+    """W x; `cast` rounds what goes into the product and what comes out of it (a model of 16-bit activations)."""
+    return cast(cast(x) @ weight.T)
+
+
+def latent_attention(h, w, p, mix, eps, shared=None, cast=exact):
     """h (T, C) -> (output (T, C), (latents, rotated key part)).  `shared`: the pair of another layer."""
     T = h.shape[0]
     H, dim, rd, vd, rank = mix["heads"], mix["dim"], mix["rot_dim"], mix["vdim"], mix["kv_rank"]
     pos = np.arange(T)
-    cq = rms_norm(h @ w[p + "dq"].T, w[p + "dq.norm"], eps)
-    q = (cq @ w[p + "uq"].T).reshape(T, H, dim + rd)
+    cq = rms_norm(linear(h, w[p + "dq"], cast), w[p + "dq.norm"], eps)
+    q = linear(cq, w[p + "uq"], cast).reshape(T, H, dim + rd)
     if shared is None:
-        kv = h @ w[p + "dkv"].T
-        c = rms_norm(kv[:, :rank], w[p + "dkv.norm"], eps)
-        kr = rotate(kv[:, rank:], pos, mix["rot"])
+        kv = linear(h, w[p + "dkv"], cast)
+        c = cast(rms_norm(kv[:, :rank], w[p + "dkv.norm"], eps))
+        kr = cast(rotate(kv[:, rank:], pos, mix["rot"]))
     else:
         c, kr = shared
-    qr = rotate(q[..., dim:], pos, mix["rot"])
-    k = (c @ w[p + "uk"].T).reshape(T, H, dim)
-    v = (c @ w[p + "uv"].T).reshape(T, H, vd)
+    qr = cast(rotate(q[..., dim:], pos, mix["rot"]))
+    k = linear(c, w[p + "uk"], cast).reshape(T, H, dim)
+    v = linear(c, w[p + "uv"], cast).reshape(T, H, vd)
     qq = np.concatenate([q[..., :dim], qr], -1)
     kk = np.concatenate([k, np.repeat(kr[:, None, :], H, 1)], -1)
     o = windowed_attention(qq, kk, v, mix["scale"], mix["mask"]["size"])
-    o = o * sigmoid(h @ w[p + "g"].T)[..., None]
-    return o.reshape(T, H * vd) @ w[p + "o"].T, (c, kr)
+    o = o * sigmoid(linear(h, w[p + "g"], cast))[..., None]
+    return linear(o.reshape(T, H * vd), w[p + "o"], cast), (c, kr)
 
 
 def gla_recurrence(q, k, v, alpha, state=None):
@@ -112,25 +121,25 @@ def gla_recurrence(q, k, v, alpha, state=None):
     return o, S
 
 
-def gla(h, w, p, mix, eps):
+def gla(h, w, p, mix, eps, cast=exact):
     T = h.shape[0]
     H, D, V = mix["heads"], mix["dim"], mix["vdim"]
-    q = (h @ w[p + "q"].T).reshape(T, H, D) * D ** -0.5
-    k = (h @ w[p + "k"].T).reshape(T, H, D)
-    v = (h @ w[p + "v"].T).reshape(T, H, V)
-    z = (h @ w[p + "a1"].T) @ w[p + "a2"].T + w[p + "a2.b"]
+    q = linear(h, w[p + "q"], cast).reshape(T, H, D) * D ** -0.5
+    k = linear(h, w[p + "k"], cast).reshape(T, H, D)
+    v = linear(h, w[p + "v"], cast).reshape(T, H, V)
+    z = linear(h, w[p + "a1"], cast) @ w[p + "a2"].T + w[p + "a2.b"]
     alpha = (sigmoid(z) ** (1.0 / mix["tau"])).reshape(T, H, D)
     o, _ = gla_recurrence(q, k, v, alpha)
     o = rms_norm(o, w[p + "norm"], eps).reshape(T, H * V)
-    return (o * silu(h @ w[p + "g"].T)) @ w[p + "o"].T
+    return linear(o * silu(linear(h, w[p + "g"], cast)), w[p + "o"], cast)
 
 
-def dense_ffn(h, w, p):
-    a = silu(h @ w[p + "gate"].T + w[p + "gate.b"]) * (h @ w[p + "up"].T + w[p + "up.b"])
-    return a @ w[p + "down"].T + w[p + "down.b"]
+def dense_ffn(h, w, p, cast=exact):
+    a = silu(linear(h, w[p + "gate"], cast) + w[p + "gate.b"]) * (linear(h, w[p + "up"], cast) + w[p + "up.b"])
+    return linear(a, w[p + "down"], cast) + w[p + "down.b"]
 
 
-def forward(cfg, w, tokens, dtype=np.float64):
+def forward(cfg, w, tokens, dtype=np.float64, cast=exact):
     """(logits (T, V), residual stream after every layer (L, T, C)) of one sequence."""
     w = {n: np.asarray(a, dtype) for n, a in w.items()}
     eps = cfg["norm"]["eps"]
@@ -140,16 +149,16 @@ def forward(cfg, w, tokens, dtype=np.float64):
         p, mix = f"l{i}.", layer["mixer"]
         h = layer_norm(x, w[p + "norm1"], eps)
         if layer["type"] == "gla":
-            y = gla(h, w, p + "mix.", mix, eps)
+            y = gla(h, w, p + "mix.", mix, eps, cast)
         elif layer["type"] == "latent_attention":
             src = mix.get("kv_from")
-            y, kv = latent_attention(h, w, p + "mix.", mix, eps, None if src is None else kept[src])
+            y, kv = latent_attention(h, w, p + "mix.", mix, eps, None if src is None else kept[src], cast)
             kept[i] = kv
         else:
             raise ValueError(layer["type"])
         x = x + layer_norm(y, w[p + "norm1b"], eps)
         if layer["mlp"] is not None:
-            y = dense_ffn(layer_norm(x, w[p + "norm2"], eps), w, p + "mlp.")
+            y = dense_ffn(layer_norm(x, w[p + "norm2"], eps), w, p + "mlp.", cast)
             x = x + layer_norm(y, w[p + "norm2b"], eps)
         stream.append(x)
-    return layer_norm(x, w["final.norm"], eps) @ w["head"].T, np.stack(stream)
+    return cast(layer_norm(x, w["final.norm"], eps)) @ w["head"].T, np.stack(stream)
