@@ -179,6 +179,9 @@ def kernels(width: int, ff: int, T: int, window: int) -> list[dict]:
     add(f"residual_norm {T}x{C}", "add_rmsnorm", us, T * C * 14.0)
     us = graph_us([lambda s=s: ops.add_rmsnorm(s[0], s[1], w, 1e-6, s[3]) for s in xs])
     add(f"add_rmsnorm {T}x{C}", "itself", us, T * C * 16.0)
+    few = int(T * (att.q_rank + 576) * 4 / (C * 16))             # as many bytes as latent_prepare moves
+    us = graph_us([lambda s=s: ops.add_rmsnorm(s[0][:few], s[1][:few], w, 1e-6, s[3][:few]) for s in xs])
+    add(f"add_rmsnorm {few}x{C}", "itself", us, few * C * 16.0)
     del xs
 
     # ---- decode: matvecs
@@ -239,6 +242,11 @@ def kernels(width: int, ff: int, T: int, window: int) -> list[dict]:
     qkv1, o1 = torch.randn(1, 3 * C, device=dev), torch.empty(1, C, device=dev)
     us = graph_us([lambda s=s: ops.decode_attention_rope(qkv1, cs, cs, pos, s[0], s[1], o1, 0) for s in kvs])
     add(f"decode_attention_rope {H} heads, {T + 1} keys", "itself", us, (T + 1) * C * 8.0)
+    # the same kernel over as many bytes as the two mixers above move
+    for keys in (int((min(window, T + 1) * 576 * 2.0 + 2.0 * att.n_kv * 512) / (C * 8)), int(H * hd * hd / C)):
+        few = torch.full((1,), keys - 1, dtype=torch.long, device=dev)
+        us = graph_us([lambda s=s: ops.decode_attention_rope(qkv1, cs, cs, few, s[0], s[1], o1, 0) for s in kvs])
+        add(f"decode_attention_rope {H} heads, {keys} keys", "itself", us, keys * C * 8.0)
     return rows
 
 

@@ -589,7 +589,10 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
     }
   }
   __syncthreads();
+  // the values, the gate and the norm's weights take the place of the state and the factors
   stage_rows(sm.shi, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  stage_rows(sm.slo, VD + 8, base + p.g_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  for (int i = tid; i < VD; i += kGmThreads) sm.fac[i] = i < p.vdim ? p.norm_w[i] : 0.f;
   stage_wait();
   __syncthreads();
 #pragma unroll
@@ -629,20 +632,21 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
     const int t = half ? rb : ra;
     if (t >= cnt) continue;
     const float inv = 1.0f / sqrtf((half ? sb : sa) / (float)p.vdim + p.eps);
-    const bf16* g = base + (size_t)t * p.ldp + p.g_off + h * p.vdim;
+    const bf16* g = sm.slo + t * (VD + 8);
     bf16* out = reinterpret_cast<bf16*>(p.out) + (size_t)(b * p.T + t0 + t) * p.ldo + h * p.vdim;
 #pragma unroll
     for (int i = 0; i < VD / 8; ++i) {
       const int v = i * 8 + c2;
+      const uint32_t gg = *reinterpret_cast<const uint32_t*>(g + v);
+      const float2 nw = *reinterpret_cast<const float2*>(sm.fac + v);
+      const float gx = bf_lo(gg), gy = bf_hi(gg);
+      const float x = o[i][2 * half] * inv * nw.x * __fdividef(gx, 1.f + __expf(-gx));
+      const float y = o[i][2 * half + 1] * inv * nw.y * __fdividef(gy, 1.f + __expf(-gy));
       if (vec) {
-        if (v < p.vdim) {
-          const uint32_t gg = *reinterpret_cast<const uint32_t*>(g + v);
-          *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(o[i][2 * half] * inv * p.norm_w[v] * silu_f(bf_lo(gg)),
-                                                            o[i][2 * half + 1] * inv * p.norm_w[v + 1] * silu_f(bf_hi(gg)));
-        }
+        if (v < p.vdim) *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(x, y);
       } else {
-        if (v < p.vdim) out[v] = from_f<bf16>(o[i][2 * half] * inv * p.norm_w[v] * silu_f(to_f(g[v])));
-        if (v + 1 < p.vdim) out[v + 1] = from_f<bf16>(o[i][2 * half + 1] * inv * p.norm_w[v + 1] * silu_f(to_f(g[v + 1])));
+        if (v < p.vdim) out[v] = from_f<bf16>(x);
+        if (v + 1 < p.vdim) out[v + 1] = from_f<bf16>(y);
       }
     }
   }
@@ -794,7 +798,7 @@ template <typename T> static int gla_prefill(const nb_gla_args& a, const GlaWs& 
 template <int VD> static int gla_prefill_mma(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
   const int chunks = gla_chunks(a.T), subs = (a.T + kGS - 1) / kGS, dt = (a.dim + 63) / 64, HD = a.H * a.dim;
   const int vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ldp % 8 == 0 && a.q_off % 8 == 0 && a.k_off % 8 == 0 && a.v_off % 8 == 0 &&
-                  a.g_off % 2 == 0 && a.ldo % 2 == 0 && (uintptr_t)a.p % 16 == 0 && (uintptr_t)a.out % 4 == 0;
+                  a.g_off % 8 == 0 && a.ldo % 2 == 0 && (uintptr_t)a.p % 16 == 0 && (uintptr_t)a.out % 4 == 0;
   static bool done[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);

@@ -462,7 +462,7 @@ __global__ void __launch_bounds__(kTThreads) latent_attention_bf16_kernel(const 
 // and as values from there.  Everything that does not depend on the launch before — the rows of earlier positions, the
 // weights — is requested ahead of the dependency wait.
 constexpr int kLdThreads = 256, kLdWarps = kLdThreads / 32;
-constexpr int kLdCols = 4;             // column pairs per thread: rank <= 2 * 256 * 4
+constexpr int kLdCols = 2;             // groups of four columns per thread: rank <= 4 * 256 * 2
 constexpr int kLdPre = 16;             // W_uk words a thread may hold ahead of the wait
 
 __device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
@@ -478,14 +478,18 @@ template <> __device__ __forceinline__ float dot16<float>(const void* r, const f
   const float4 t = *reinterpret_cast<const float4*>(r), a = *reinterpret_cast<const float4*>(q);
   return t.x * a.x + t.y * a.y + t.z * a.z + t.w * a.w;
 }
-__device__ __forceinline__ float2 pair_at(const bf16* r) {
-  const uint32_t t = *reinterpret_cast<const uint32_t*>(r);
-  return make_float2(bf_lo(t), bf_hi(t));
+__device__ __forceinline__ float4 quad_at(const bf16* r) {
+  const uint2 t = *reinterpret_cast<const uint2*>(r);
+  return make_float4(bf_lo(t.x), bf_hi(t.x), bf_lo(t.y), bf_hi(t.y));
 }
-__device__ __forceinline__ float2 pair_at(const float* r) { return *reinterpret_cast<const float2*>(r); }
+__device__ __forceinline__ float4 quad_at(const float* r) { return *reinterpret_cast<const float4*>(r); }
 
-// Elements between staged rows: an odd number of 16-byte pieces, so that eight rows sit on different banks.
-template <typename T> __host__ __device__ inline int staged_row(int rdp) { return rdp % (32 / (int)sizeof(T)) ? rdp : rdp + 16 / (int)sizeof(T); }
+// Elements between staged rows: 4 modulo 8 pieces of 16 bytes, so that two keys' four lanes each read eight different
+// groups of banks.
+template <typename T> __host__ __device__ inline int staged_row(int rdp) {
+  const int per = 16 / (int)sizeof(T), pieces = rdp / per;
+  return (pieces + ((4 - pieces % 8 + 8) & 7)) * per;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_latent_decode_args p, int stage) {
@@ -500,9 +504,9 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   float* qn = ol + rdp;                // [dk] this head's query
   float* cs = qn + ((dk + 7) & ~7);    // [rot] the position's rotary entries
   float* sn = cs + ((p.rot + 7) & ~7);
-  float* part = sn + ((p.rot + 7) & ~7);   // [kLdThreads * 2] partial sums
+  float* part = sn + ((p.rot + 7) & ~7);   // [kLdThreads * 4] partial sums
   const int pairs = (p.rank + 1) / 2, pper = (pairs + S - 1) / S, slot = (2 * pper + 2 + 3) & ~3;
-  float* xch = part + 2 * kLdThreads;  // [S][slot] what the CTAs send: their part of this CTA's slice, maximum, sum
+  float* xch = part + 4 * kLdThreads;  // [S][slot] what the CTAs send: their part of this CTA's slice, maximum, sum
   float* sc = xch + S * slot;          // [stage] scores, then weights, of the staged keys
   T* rows = reinterpret_cast<T*>(sc + ((stage + 3) & ~3));   // [stage][ldr]
 
@@ -543,18 +547,25 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
     prefetch_l2(uv + (size_t)(v0 + v) * p.ldu + c * 64);
   }
   // the position's rotary entries and the norm's weights
-  for (int i = tid; i < p.rot; i += kLdThreads) { cs[i] = p.cos2[(size_t)pos * p.rot + i]; sn[i] = p.sin2[(size_t)pos * p.rot + i]; }
+  const float* ct = p.cos2 + (size_t)pos * p.rot;
+  const float* stb = p.sin2 + (size_t)pos * p.rot;
+  const float c_pre = tid < p.rot ? ct[tid] : 0.f, s_pre = tid < p.rot ? stb[tid] : 0.f;
   const int mine = (int)pos - k0;      // this position's place among this CTA's keys, if 0 <= mine < cnt
   const bool holds = mine >= 0 && mine < cnt;
-  constexpr int kKv = 2 * kLdCols;     // elements of the position's latent per thread
+  constexpr int kKv = 4 * kLdCols;     // elements of the position's latent per thread
   float kvw[kKv], kvv[kKv];
   if (p.kv_off >= 0 && holds) {
 #pragma unroll
     for (int u = 0; u < kKv; ++u) kvw[u] = tid + u * kLdThreads < p.rank ? p.kv_norm[tid + u * kLdThreads] : 0.f;
   }
+  for (int j = stage + warp; j < cnt; j += kLdWarps)     // rows that are staged later: on their way to L2
+    for (int c = lane * (64 / (int)sizeof(T)) * 2; c < rd; c += 32 * (64 / (int)sizeof(T)) * 2)
+      prefetch_l2(cache + (size_t)(k0 + j) * p.ldc + c);
   cluster.barrier_arrive();
 
   pdl_enter();
+  if (tid < p.rot) { cs[tid] = c_pre; sn[tid] = s_pre; }
+  for (int i = tid + kLdThreads; i < p.rot; i += kLdThreads) { cs[i] = ct[i]; sn[i] = stb[i]; }
   for (int i = tid; i < dk; i += kLdThreads) qn[i] = p.q[(size_t)b * p.ldq + h * dk + i];
   const float gate = p.a[(size_t)b * p.lda + p.g_off + h];
   for (int i = rd + tid; i < rdp; i += kLdThreads) qa[i] = 0.f;
@@ -633,12 +644,13 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   cluster.sync();
 
   // softmax and weighted latent over the staged rows.  Scores: four lanes share a key, sixteen bytes at a time.  Latent: a
-  // thread owns up to kLdCols column pairs, or, with few columns, one pair of every `groups`-th key.
-  const int wcols = min(pairs, kLdThreads), groups = pairs <= kLdThreads ? kLdThreads / wcols : 1, gi = tid / wcols, wc = tid - gi * wcols;
+  // thread owns four columns (or kLdCols times four); with few columns the keys are split over `groups` of threads.
+  const int quads = (p.rank + 3) / 4;
+  const int wcols = min(quads, kLdThreads), groups = quads <= kLdThreads ? kLdThreads / wcols : 1, gi = tid / wcols, wc = tid - gi * wcols;
   float m = -FLT_MAX, l = 0.f;
-  float2 acc[kLdCols];
+  float4 acc[kLdCols];
 #pragma unroll
-  for (int u = 0; u < kLdCols; ++u) acc[u] = make_float2(0.f, 0.f);
+  for (int u = 0; u < kLdCols; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int base = 0; base < cnt; base += stage) {
     const int nk = min(stage, cnt - base);
     if (base > 0) {
@@ -654,6 +666,7 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
       float s = 0.f;
       if (j < nk) {
         const T* r = rows + (size_t)j * ldr;
+#pragma unroll 6
         for (int c = lane & 3; c < pieces; c += 4) s += dot16<T>(r + c * kPiece, qa + c * kPiece);
       }
       s += __shfl_xor_sync(0xffffffffu, s, 1);
@@ -681,15 +694,17 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
     l = l * corr + block_sum<kLdWarps>(sum, red3);   // its barrier also publishes the weights
 #pragma unroll
     for (int u = 0; u < kLdCols; ++u) {
-      acc[u].x *= corr; acc[u].y *= corr;
+      acc[u].x *= corr; acc[u].y *= corr; acc[u].z *= corr; acc[u].w *= corr;
       const int c = wc + u * kLdThreads;
-      if (gi < groups && c < pairs) {
+      if (gi < groups && c < quads) {
 #pragma unroll 8
         for (int j = gi; j < nk; j += groups) {
           const float w = sc[j];
-          const float2 t = pair_at(rows + (size_t)j * ldr + 2 * c);
+          const float4 t = quad_at(rows + (size_t)j * ldr + 4 * c);   // columns past the latent: never sent
           acc[u].x = fmaf(w, t.x, acc[u].x);
           acc[u].y = fmaf(w, t.y, acc[u].y);
+          acc[u].z = fmaf(w, t.z, acc[u].z);
+          acc[u].w = fmaf(w, t.w, acc[u].w);
         }
       }
     }
@@ -697,14 +712,14 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   // every CTA sends the parts of its weighted latent to the CTAs that merge them: slice r (2 * pper columns) to CTA r
 #pragma unroll
   for (int u = 0; u < kLdCols; ++u) {
-    if (u * kLdThreads < pairs) {      // block-uniform
-      part[2 * tid] = acc[u].x; part[2 * tid + 1] = acc[u].y;
+    if (u * kLdThreads < quads) {      // block-uniform
+      reinterpret_cast<float4*>(part)[tid] = acc[u];
       __syncthreads();
-      const int cols = min(pairs - u * kLdThreads, kLdThreads);
-      for (int i = tid; i < 2 * cols; i += kLdThreads) {
+      const int cols = min(4 * kLdThreads, p.rank - 4 * u * kLdThreads);
+      for (int i = tid; i < cols; i += kLdThreads) {
         float v = 0.f;
-        for (int g = 0; g < groups; ++g) v += part[2 * g * wcols + i];
-        const int col = 2 * u * kLdThreads + i, to = col / (2 * pper);
+        for (int g = 0; g < groups; ++g) v += part[4 * g * wcols + i];
+        const int col = 4 * u * kLdThreads + i, to = col / (2 * pper);
         cluster.map_shared_rank(xch, to)[rank_id * slot + col - to * 2 * pper] = v;
       }
       __syncthreads();
@@ -875,14 +890,14 @@ extern "C" int nb_latent_decode(const nb_latent_decode_args* a, void* stream) {
   if ((uintptr_t)a->cache % 16 || a->ldc % 8 || (uintptr_t)a->uk % 16 || (uintptr_t)a->uv % 16 || a->ldu % 8) return NB_ERR_ALIGN;
   if (a->H > 65535 || a->B > 65535) return NB_ERR_SHAPE;
   if (int rc = check_device()) return rc;
-  if (a->rank > 2 * kLdThreads * kLdCols) return NB_ERR_SHAPE;
+  if (a->rank > 4 * kLdThreads * kLdCols) return NB_ERR_SHAPE;
   const int want = 592 / std::max(1, a->B * a->H), S = want >= 8 ? 8 : want >= 4 ? 4 : want >= 2 ? 2 : 1;
   const int most = a->window > 0 ? std::min(a->window, a->ctx) : a->ctx;
   const int wide = a->cache_dtype == NB_F32;
   const int rdp = (a->rank + a->rot + 7) & ~7;
   const size_t row = (size_t)(wide ? staged_row<float>(rdp) * 4 : staged_row<bf16>(rdp) * 2);
   const int pper = ((a->rank + 1) / 2 + S - 1) / S, slot = (2 * pper + 2 + 3) & ~3;
-  const size_t fixed = ((size_t)2 * rdp + ((a->dim + a->rot + 7) & ~7) + 2 * ((a->rot + 7) & ~7) + 2 * kLdThreads + S * slot + 4) * 4;
+  const size_t fixed = ((size_t)2 * rdp + ((a->dim + a->rot + 7) & ~7) + 2 * ((a->rot + 7) & ~7) + 4 * kLdThreads + S * slot + 4) * 4;
   if (fixed + 8 * (row + 4) > kLatentMaxSmem) return NB_ERR_SHAPE;
   // as many of a CTA's rows at a time as shared memory holds; two CTAs per SM when they do not all fit one each
   const size_t budget = (size_t)a->B * a->H * S > 112 && fixed + 8 * (row + 4) <= kLatentHalfSmem ? kLatentHalfSmem : kLatentMaxSmem;
