@@ -484,11 +484,15 @@ __device__ __forceinline__ float4 quad_at(const bf16* r) {
 }
 __device__ __forceinline__ float4 quad_at(const float* r) { return *reinterpret_cast<const float4*>(r); }
 
-// Elements between staged rows: 4 modulo 8 pieces of 16 bytes, so that two keys' four lanes each read eight different
-// groups of banks.
-template <typename T> __host__ __device__ inline int staged_row(int rdp) {
-  const int per = 16 / (int)sizeof(T), pieces = rdp / per;
-  return (pieces + ((4 - pieces % 8 + 8) & 7)) * per;
+// Sixteen bytes of a staged row times the matching part of the query.
+__device__ __forceinline__ float dot_piece(const bf16* r, const float (&q)[8]) {
+  const uint4 t = *reinterpret_cast<const uint4*>(r);
+  return (bf_lo(t.x) * q[0] + bf_hi(t.x) * q[1]) + (bf_lo(t.y) * q[2] + bf_hi(t.y) * q[3]) + (bf_lo(t.z) * q[4] + bf_hi(t.z) * q[5]) +
+         (bf_lo(t.w) * q[6] + bf_hi(t.w) * q[7]);
+}
+__device__ __forceinline__ float dot_piece(const float* r, const float (&q)[4]) {
+  const float4 t = *reinterpret_cast<const float4*>(r);
+  return (t.x * q[0] + t.y * q[1]) + (t.z * q[2] + t.w * q[3]);
 }
 
 template <typename T>
@@ -498,7 +502,7 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   cg::cluster_group cluster = cg::this_cluster();
   const int S = (int)cluster.num_blocks(), rank_id = (int)cluster.block_rank();
   const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int rd = p.rank + p.rot, dk = p.dim + p.rot, rdp = (rd + 7) & ~7, ldr = staged_row<T>(rdp);
+  const int rd = p.rank + p.rot, dk = p.dim + p.rot, rdp = (rd + 7) & ~7, ldr = rdp;
   float* qa = dsm;                     // [rdp] q' and the rotated query part: what the cached rows are multiplied with
   float* ol = qa + rdp;                // [rdp] merged latent
   float* qn = ol + rdp;                // [dk] this head's query
@@ -643,7 +647,9 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   if (pn == 0) cluster.barrier_wait();
   cluster.sync();
 
-  // softmax and weighted latent over the staged rows.  Scores: four lanes share a key, sixteen bytes at a time.  Latent: a
+  // softmax and weighted latent over the staged rows.  Scores: a warp takes four
+  // keys at a time, a lane holds its part of the query in registers (shared-memory reads of the query would cost more than
+  // those of the rows).  Latent: a
   // thread owns four columns (or kLdCols times four); with few columns the keys are split over `groups` of threads.
   const int quads = (p.rank + 3) / 4;
   const int wcols = min(quads, kLdThreads), groups = quads <= kLdThreads ? kLdThreads / wcols : 1, gi = tid / wcols, wc = tid - gi * wcols;
@@ -651,6 +657,16 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
   float4 acc[kLdCols];
 #pragma unroll
   for (int u = 0; u < kLdCols; ++u) acc[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+  constexpr int kQp = sizeof(T) == 2 ? 3 : 5;
+  float qreg[kQp][kPiece];
+#pragma unroll
+  for (int x = 0; x < kQp; ++x)
+#pragma unroll
+    for (int e = 0; e < kPiece; e += 4) {
+      const int c = x * 32 + lane;
+      const float4 v = c < pieces ? *reinterpret_cast<const float4*>(qa + c * kPiece + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      qreg[x][e] = v.x; qreg[x][e + 1] = v.y; qreg[x][e + 2] = v.z; qreg[x][e + 3] = v.w;
+    }
   for (int base = 0; base < cnt; base += stage) {
     const int nk = min(stage, cnt - base);
     if (base > 0) {
@@ -661,20 +677,33 @@ __global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const nb_l
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     float mx = -FLT_MAX;
-    for (int j0 = warp * 8; j0 < nk; j0 += kLdWarps * 8) {
-      const int j = j0 + (lane >> 2);
-      float s = 0.f;
-      if (j < nk) {
-        const T* r = rows + (size_t)j * ldr;
-#pragma unroll 6
-        for (int c = lane & 3; c < pieces; c += 4) s += dot16<T>(r + c * kPiece, qa + c * kPiece);
+    for (int j0 = warp * 4; j0 < nk; j0 += kLdWarps * 4) {
+      float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int x = 0; x < kQp; ++x) {
+        const int c = x * 32 + lane;
+        if (c < pieces) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) s[k] += dot_piece(rows + (size_t)min(j0 + k, nk - 1) * ldr + c * kPiece, qreg[x]);
+        }
       }
-      s += __shfl_xor_sync(0xffffffffu, s, 1);
-      s += __shfl_xor_sync(0xffffffffu, s, 2);
-      s *= p.scale;
+      for (int c = kQp * 32 + lane; c < pieces; c += 32)       // wider rows than the registers hold
+#pragma unroll
+        for (int k = 0; k < 4; ++k) s[k] += dot16<T>(rows + (size_t)min(j0 + k, nk - 1) * ldr + c * kPiece, qa + c * kPiece);
+      // four sums over the warp: lanes keep one key each from the second halving on
+      const bool hi16 = lane & 16, hi8 = lane & 8;
+      float a = hi16 ? s[2] : s[0], b2 = hi16 ? s[3] : s[1];
+      a += __shfl_xor_sync(0xffffffffu, hi16 ? s[0] : s[2], 16);
+      b2 += __shfl_xor_sync(0xffffffffu, hi16 ? s[1] : s[3], 16);
+      float t = hi8 ? b2 : a;
+      t += __shfl_xor_sync(0xffffffffu, hi8 ? a : b2, 8);
+#pragma unroll
+      for (int x = 4; x > 0; x >>= 1) t += __shfl_xor_sync(0xffffffffu, t, x);
+      t *= p.scale;
+      const int j = j0 + (hi16 ? 2 : 0) + (hi8 ? 1 : 0);
       if (j < nk) {
-        if ((lane & 3) == 0) sc[j] = s;
-        mx = fmaxf(mx, s);
+        if ((lane & 7) == 0) sc[j] = t;
+        mx = fmaxf(mx, t);
       }
     }
     mx = warp_max(mx);
@@ -895,7 +924,7 @@ extern "C" int nb_latent_decode(const nb_latent_decode_args* a, void* stream) {
   const int most = a->window > 0 ? std::min(a->window, a->ctx) : a->ctx;
   const int wide = a->cache_dtype == NB_F32;
   const int rdp = (a->rank + a->rot + 7) & ~7;
-  const size_t row = (size_t)(wide ? staged_row<float>(rdp) * 4 : staged_row<bf16>(rdp) * 2);
+  const size_t row = (size_t)rdp * (wide ? 4 : 2);
   const int pper = ((a->rank + 1) / 2 + S - 1) / S, slot = (2 * pper + 2 + 3) & ~3;
   const size_t fixed = ((size_t)2 * rdp + ((a->dim + a->rot + 7) & ~7) + 2 * ((a->rot + 7) & ~7) + 4 * kLdThreads + S * slot + 4) * 4;
   if (fixed + 8 * (row + 4) > kLatentMaxSmem) return NB_ERR_SHAPE;
