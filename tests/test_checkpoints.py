@@ -49,6 +49,34 @@ def test_torch_nbpack_loader_structure_on_cpu(name, bs):
 
 
 @pytest.mark.gpu
+def test_a_packed_model_folder_runs_through_the_registry(built_lib, tmp_path):
+    """The registry loads a packed decoder from a folder; its session takes portions of a prompt and single tokens from the
+    same call as the layered models' and agrees with the reference's logits."""
+    import json
+    import shutil
+    from nativebit_b200 import registry
+    exp = np.load(os.path.join(GOLD, "tiny_nbpack_npz_expected.npz"))
+    cfg = {k: getattr(_Cfg, k) for k in ("vocab_size", "n_layers", "n_embd", "n_head", "ffn_hidden", "context_len")}
+    (tmp_path / "config.json").write_text(json.dumps({"architecture": "PackedGPT", **cfg}))
+    shutil.copy(os.path.join(GOLD, "tiny.nbpack.npz"), tmp_path / "model.nbpack.npz")
+    with pytest.raises(registry.UnsupportedDtype):
+        registry.load_model(str(tmp_path), "float32")
+    model = registry.load_model(str(tmp_path), "bfloat16")
+    s = registry.open_session(model)
+    prompt, n = torch.from_numpy(exp["prompt"]).cuda(), exp["prompt"].shape[1]
+    for cuts in ([n], [2, n - 4, 1, 1]):
+        got, at = [], 0
+        for c in cuts:
+            got.append(s.extend(prompt[:, at:at + c], list(range(c)))[0].clone())
+            at += c
+        ref = exp["logits"]
+        assert np.abs(torch.cat(got).cpu().numpy() - ref).max() <= 2e-3 * np.abs(ref).max()
+        assert int(s.token[0, 0]) == int(ref[-1].argmax())
+        s.reset()
+    s.check()
+
+
+@pytest.mark.gpu
 def test_npz_checkpoint_decodes_like_the_reference(built_lib):
     from nativebit_b200 import generate as G
     dev = torch.device("cuda:0")
