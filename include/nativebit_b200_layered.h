@@ -16,26 +16,46 @@ extern "C" {
 #endif
 
 typedef enum { NB_NORM_RMS = 0, NB_NORM_LAYER = 1 } nb_norm;   /* LAYER: mean taken off, weight, no bias */
-typedef enum { NB_ACT_NONE = 0, NB_ACT_SWIGLU_PAIRS = 1 } nb_act;
-/* NB_ACT_SWIGLU_PAIRS: rows 2i and 2i + 1 of the weight are gate and up of channel i; y has N / 2 columns,
- * silu(gate + bias) * (up + bias). */
+typedef enum { NB_ACT_NONE = 0, NB_ACT_SWIGLU_PAIRS = 1, NB_ACT_CLAMPED_GLU_PAIRS = 2 } nb_act;
+/* .._PAIRS: rows 2i and 2i + 1 of the weight are gate and up of channel i (g = gate + bias, u = up + bias); y has N / 2
+ * columns.  SWIGLU: silu(g) * u.  CLAMPED_GLU: g = min(g, limit), u clamped to +-limit, g * sigmoid(alpha * g) * (u + 1)
+ * (alpha and limit are not read by the other activations). */
 
-/* ---- x (rows, C) fp32 = table[token] * scale for a bf16 (V, C) table; token ids are clamped to [0, V). */
-int nb_embed_scaled(const void* table_bf16, const int64_t* token, int rows, int V, int C, float scale, float* x, void* stream);
+/* ---- x (rows, streams, C) fp32 = table[token] * scale, once per stream, for a bf16 (V, C) table; token ids are clamped
+ * to [0, V). */
+int nb_embed_scaled(const void* table_bf16, const int64_t* token, int rows, int V, int C, float scale, int streams, float* x, void* stream);
 
 /* ---- one step of the residual chain, per row: x += norm(y) * wy (if y), then h = norm(x) * w (if h).
  * x, y (rows, C) fp32; h (rows, ldh) of h_dtype. */
 int nb_residual_norm(float* x, const float* y, const float* wy, const float* w, int norm, float eps, void* h, int h_dtype, int ldh,
                      int rows, int C, void* stream);
 
+/* ---- hyper-connections: a residual of `streams` vectors per row, mixed at every sublayer.  With the result y of the
+ * sublayer before (the sum of one or two branches, each through an optional norm of its own and times its weight; none if
+ * y0 is NULL), per row:
+ *   x_out_t = sum_s mix[s][t] x_s + share_t * y        the streams behind it (not written if x_out is NULL)
+ *   u       = sum_s read_s x_s + direct * y            what the next sublayer reads: its weights applied to those streams
+ *   h       = norm(u) * norm_w
+ * coef: fp32 [read (streams) | direct | share (streams) | mix (streams, streams)].  x, x_out (rows, streams, C), y (rows, C).
+ * nb_stream_norm: many rows, h (rows, ldh) of h_dtype; x_out may be x. */
+enum { NB_MAX_STREAMS = 8 };
+typedef struct {
+  const float* x;
+  float* x_out;
+  const float *y0, *w0, *y1, *w1, *coef, *norm_w;
+  float eps;
+  int streams, C, y_norm, norm;   /* y_norm: nb_norm, or -1 for none */
+} nb_stream_args;
+int nb_stream_norm(const nb_stream_args* a, void* h, int h_dtype, int ldh, int rows, void* stream);
+
 /* ---- y (M, N) = x (M, K) . w (N, K)^T (+ bias) for many rows.
  * nb_linear_bf16: bf16 x on the tcgen05 tensor cores, fp32 accumulation, y NB_BF16 or NB_F32; x and w 16-byte
  * aligned, ldx and ldw multiples of 8; `status`: device int, NB_ERR_TIMEOUT if a bounded wait ran out, or NULL.
  * nb_linear_f32: fp32 x and y, fp32 multiply-adds. */
-int nb_linear_bf16(const void* x, int ldx, const void* w, int ldw, const float* bias, int act, int M, int N, int K, void* y, int y_dtype,
-                   int ldy, int* status, void* stream);
-int nb_linear_f32(const float* x, int ldx, const void* w, int ldw, const float* bias, int act, int M, int N, int K, float* y, int ldy,
-                  void* stream);
+int nb_linear_bf16(const void* x, int ldx, const void* w, int ldw, const float* bias, int act, float alpha, float limit, int M, int N, int K,
+                   void* y, int y_dtype, int ldy, int* status, void* stream);
+int nb_linear_f32(const float* x, int ldx, const void* w, int ldw, const float* bias, int act, float alpha, float limit, int M, int N, int K,
+                  float* y, int ldy, void* stream);
 
 /* ---- y (N) = w (N, K) . act for ONE row (decode), fp32 activations, with the element-wise step in front folded in:
  *   norm_w NULL:            act = x
@@ -51,10 +71,15 @@ typedef struct {
   const float* delta_w; /* K or NULL */
   float* x_out;         /* K or NULL */
   const float* norm_w;  /* K or NULL */
-  float eps;
+  float eps, alpha, limit;
   int N, K, ldw, act, norm;
 } nb_matvec_args;
 int nb_matvec_bf16(const nb_matvec_args* a, void* stream);
+/* The same behind hyper-connections: act = the h of nb_stream_norm for one row (s->x_out != s->x); of `a` the launch reads
+ * w, bias, y, N, K, ldw and the activation. */
+int nb_matvec_streams(const nb_matvec_args* a, const nb_stream_args* s, void* stream);
+/* Two products of plain rows (no norm, no delta) in one launch. */
+int nb_matvec_pair(const nb_matvec_args* a, const nb_matvec_args* b, void* stream);
 
 /* ---- latent attention -------------------------------------------------------------------------------------
  * Cache of a layer: (B, ctx, ldc) rows [latent (rank) | rotated key part (rot)] of the activation dtype, ldc a
@@ -108,11 +133,53 @@ typedef struct {
 } nb_latent_decode_args;
 int nb_latent_decode(const nb_latent_decode_args* a, void* stream);
 
+/* ---- grouped attention with scores mixed across heads ---------------------------------------------------------
+ * Cache of a layer: (B, ctx, ldc) rows [keys of the G heads (G * dim) | .. | values from v_off (G * vdim)] of the activation
+ * dtype, ldc and v_off multiples of 8.  Query head h reads key/value head h / (H / G).  Per query i and key j of the window
+ * (0 <= i - j < window): s_h = softcap * tanh(q_h . k * scale / softcap) - penalty[h][i - j], then s'_h = sum_g talk[h][g] s_g,
+ * softmax of s'_h over the keys, out_h = sum of values * sigmoid(gate), the gate per element.  softcap <= 0: no cap;
+ * penalty NULL: none; gate NULL (g_off < 0): none.  penalty: (H, n_pen) fp32 with n_pen >= min(window, ctx); talk (H, H).
+ *
+ * nb_cache_append: cache[b][pos0 + t][0 .. cols) = src row b * T + t, columns off .. (16 bytes at a time: off and both row
+ * strides are multiples of 8, the row's last eight columns are copied whole).
+ * nb_talk_attention: T new positions pos0 .. whose keys and values are in the cache.  NB_BF16 runs on the tensor cores
+ * (scores, mixing and softmax in fp32; the softmax weights enter the second product as two bf16 terms), NB_F32 in fp32
+ * multiply-adds.  The mixed scores of a block of queries pass through the workspace (any size from
+ * nb_talk_attention_workspace_bytes(.., 1) on; with more, more queries at a time).
+ * nb_talk_decode: one new position per sequence from fp32 projections p: appends its keys and values (p at k_off, in the
+ * cache row's layout) and attends, a cluster of CTAs per sequence.  Does nothing when *pos is outside [0, ctx). */
+typedef struct {
+  const void *q, *cache, *gate;
+  void* out;
+  const float *penalty, *talk;
+  float scale, softcap;
+  int dtype, B, T, H, G, dim, vdim, ctx, ldc, v_off, ldq, ldg, ldo, pos0, window, n_pen;
+} nb_talk_attention_args;
+int nb_cache_append(const void* src, int ld, int off, int cols, void* cache, int ldc, int dtype, int B, int T, int ctx, int pos0, void* stream);
+size_t nb_talk_attention_workspace_bytes(int B, int T, int H, int pos0, int window, int query_tiles);
+int nb_talk_attention(const nb_talk_attention_args* a, void* workspace, size_t workspace_bytes, void* stream);
+
+typedef struct {
+  const float* p;
+  void* cache;
+  const float *penalty, *talk;
+  const int64_t* pos;
+  float* out;
+  float scale, softcap;
+  int cache_dtype, B, H, G, dim, vdim, ctx, ldc, v_off, ldp, q_off, k_off, g_off, ldo, window, n_pen;
+} nb_talk_decode_args;
+int nb_talk_decode(const nb_talk_decode_args* a, void* stream);
+
 /* ---- gated linear attention -------------------------------------------------------------------------------
  * p: (B * T, ldp) projections, q at q_off (H * dim), k at k_off, v at v_off (H * vdim), g at g_off, a at a_off
  * (a_rank); decay alpha = sigmoid(a2 . a + a2_b)^(1 / tau) per key channel; per head S <- diag(alpha) S + k v^T,
  * o = S^T (q * dim^-1/2); out (B * T, ldo) = RMSNorm(o) * norm_w * silu(g).  state: (B, H, dim, lds) fp32, lds a
  * multiple of 4, columns vdim .. lds zero; read and updated.
+ * kind NB_GLA_FORGET: the decay decides what is written as well.  z = p at k_off (H * dim) + a2_b, alpha = lower +
+ * (1 - lower) sigmoid(z), k = 1 - alpha, o = S^T silu(q) without a scale; no low-rank projection (a2, a_off and a_rank are
+ * not read, nor is tau) and, with g_off < 0, no output gate. */
+typedef enum { NB_GLA_LOW_RANK = 0, NB_GLA_FORGET = 1 } nb_gla_kind;
+/*
  * nb_gla_prefill works in chunks of 64 tokens; workspace of nb_gla_workspace_bytes().
  * nb_gla_decode: one token per sequence, fp32 p and out. */
 typedef struct {
@@ -120,9 +187,9 @@ typedef struct {
   void* out;
   float* state;
   const void* a2;      /* bf16 (H * dim, lda2) */
-  const float *a2_b, *norm_w;
+  const float *a2_b, *norm_w, *lower;
   float tau, eps;
-  int dtype, B, T, H, dim, vdim, ldp, q_off, k_off, v_off, g_off, a_off, a_rank, lda2, lds, ldo;
+  int kind, dtype, B, T, H, dim, vdim, ldp, q_off, k_off, v_off, g_off, a_off, a_rank, lda2, lds, ldo;
 } nb_gla_args;
 size_t nb_gla_workspace_bytes(int B, int T, int H, int dim, int vdim);
 int nb_gla_prefill(const nb_gla_args* a, void* workspace, size_t workspace_bytes, void* stream);

@@ -104,28 +104,40 @@ def _struct(name: str, pointers: str, floats: str, ints: str):
     return type(name, (_c.Structure,), {"_fields_": fields})
 
 
-MatvecArgs = _struct("MatvecArgs", "w bias y x delta delta_w x_out norm_w", "eps", "N K ldw act norm")
+MatvecArgs = _struct("MatvecArgs", "w bias y x delta delta_w x_out norm_w", "eps alpha limit", "N K ldw act norm")
+StreamArgs = _struct("StreamArgs", "x x_out y0 w0 y1 w1 coef norm_w", "eps", "streams C y_norm norm")
 LatentPrepareArgs = _struct("LatentPrepareArgs", "a cq cache q_norm kv_norm cos2 sin2", "eps",
                             "dtype B T lda q_off q_rank ldcq kv_off rank rot ctx ldc pos0")
 LatentAttentionArgs = _struct("LatentAttentionArgs", "q kv cache gate out cos2 sin2", "scale",
                               "dtype B T H dim rot vdim rank ctx ldc ldq ldkv v_off kv_rows kv_pos0 ldg ldo pos0 window")
 LatentDecodeArgs = _struct("LatentDecodeArgs", "q a cache uk uv kv_norm cos2 sin2 pos out", "scale eps",
                            "cache_dtype B H dim rot vdim rank ctx ldc ldq lda kv_off g_off ldu ldo window")
-GlaArgs = _struct("GlaArgs", "p out state a2 a2_b norm_w", "tau eps",
-                  "dtype B T H dim vdim ldp q_off k_off v_off g_off a_off a_rank lda2 lds ldo")
+GlaArgs = _struct("GlaArgs", "p out state a2 a2_b norm_w lower", "tau eps",
+                  "kind dtype B T H dim vdim ldp q_off k_off v_off g_off a_off a_rank lda2 lds ldo")
+TalkAttentionArgs = _struct("TalkAttentionArgs", "q cache gate out penalty talk", "scale softcap",
+                            "dtype B T H G dim vdim ctx ldc v_off ldq ldg ldo pos0 window n_pen")
+TalkDecodeArgs = _struct("TalkDecodeArgs", "p cache penalty talk pos out", "scale softcap",
+                         "cache_dtype B H G dim vdim ctx ldc v_off ldp q_off k_off g_off ldo window n_pen")
 
 _LAYERED_SIGNATURES = {
-    "nb_embed_scaled": (_I, [_P, _P, _I, _I, _I, _F, _P, _P]),
+    "nb_embed_scaled": (_I, [_P, _P, _I, _I, _I, _F, _I, _P, _P]),
     "nb_residual_norm": (_I, [_P, _P, _P, _P, _I, _F, _P, _I, _I, _I, _I, _P]),
-    "nb_linear_bf16": (_I, [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P, _I, _I, _P, _P]),
-    "nb_linear_f32": (_I, [_P, _I, _P, _I, _P, _I, _I, _I, _I, _P, _I, _P]),
+    "nb_stream_norm": (_I, [_c.POINTER(StreamArgs), _P, _I, _I, _I, _P]),
+    "nb_linear_bf16": (_I, [_P, _I, _P, _I, _P, _I, _F, _F, _I, _I, _I, _P, _I, _I, _P, _P]),
+    "nb_linear_f32": (_I, [_P, _I, _P, _I, _P, _I, _F, _F, _I, _I, _I, _P, _I, _P]),
     "nb_matvec_bf16": (_I, [_c.POINTER(MatvecArgs), _P]),
+    "nb_matvec_streams": (_I, [_c.POINTER(MatvecArgs), _c.POINTER(StreamArgs), _P]),
+    "nb_matvec_pair": (_I, [_c.POINTER(MatvecArgs), _c.POINTER(MatvecArgs), _P]),
     "nb_latent_prepare": (_I, [_c.POINTER(LatentPrepareArgs), _P]),
     "nb_latent_attention": (_I, [_c.POINTER(LatentAttentionArgs), _P]),
     "nb_latent_decode": (_I, [_c.POINTER(LatentDecodeArgs), _P]),
     "nb_gla_workspace_bytes": (_c.c_size_t, [_I, _I, _I, _I, _I]),
     "nb_gla_prefill": (_I, [_c.POINTER(GlaArgs), _P, _c.c_size_t, _P]),
     "nb_gla_decode": (_I, [_c.POINTER(GlaArgs), _P]),
+    "nb_cache_append": (_I, [_P, _I, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P]),
+    "nb_talk_attention_workspace_bytes": (_c.c_size_t, [_I, _I, _I, _I, _I, _I]),
+    "nb_talk_attention": (_I, [_c.POINTER(TalkAttentionArgs), _P, _c.c_size_t, _P]),
+    "nb_talk_decode": (_I, [_c.POINTER(TalkDecodeArgs), _P]),
     "nb_argmax": (_I, [_P, _I, _I, _P, _P, _P]),
 }
 

@@ -194,7 +194,7 @@ def kernels(width: int, ff: int, T: int, window: int) -> list[dict]:
         opt = dict(norm=L.NORM_LAYER, eps=1e-6, norm_w=wn, delta=d, delta_w=wn, x_out=x2) if kw in ("chain", "ffn") else \
             dict(norm=L.NORM_RMS, eps=1e-6, norm_w=wn) if kw == "rms" else {}
         if kw == "ffn":
-            opt.update(bias=bias, act=L.ACT_SWIGLU_PAIRS)
+            opt.update(bias=bias, act=L.SWIGLU)
         us = graph_us([lambda w=w: L.matvec(w, n, k, x, y, **opt) for w in ws])
         add(f"matvec_bf16 {n}x{k} ({nm})", "lm_head" if nm == "head" else "gemv_stream", us, 2.0 * n * k + 4 * (n + k))
         del ws

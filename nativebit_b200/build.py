@@ -33,7 +33,7 @@ def _nvcc() -> str:
 # library -> its sources under csrc/
 LIBRARIES = {
     "packed": (LIB_NAME, ("nb_host", "nb_unpack", "nb_gemm", "nb_gemm_fused", "nb_gemv", "nb_stream", "nb_decode", "nb_comm")),
-    "layered": (LAYERED_LIB_NAME, ("nb_host", "nb_unpack", "nb_gemm", "nb_decode", "nb_linear", "nb_latent", "nb_gla")),
+    "layered": (LAYERED_LIB_NAME, ("nb_host", "nb_unpack", "nb_gemm", "nb_decode", "nb_linear", "nb_latent", "nb_gla", "nb_talk")),
 }
 
 

@@ -52,13 +52,21 @@ struct GemmCfg {
   static constexpr int kTmemCols = 512;                  // two accumulator buffers of up to 256 columns
 };
 
-// Eight outputs silu(gate) * up from sixteen accumulator columns (gate, up, gate, up, ...) at element `at` of y.
-__device__ __forceinline__ void store_swiglu_pairs(const uint32_t (&r)[16], void* y, int y_dtype, size_t at, int count) {
+// Eight gated outputs from sixteen accumulator columns (gate, up, gate, up, ...) at element `at` of y: silu(gate) * up, or
+// the clamped form (alpha, limit).
+__device__ __forceinline__ void store_glu_pairs(const uint32_t (&r)[16], int act, float alpha, float limit, void* y, int y_dtype, size_t at,
+                                                int count) {
   float o[8];
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
-    const float g = __uint_as_float(r[2 * j]), u = __uint_as_float(r[2 * j + 1]);
-    o[j] = g / (1.0f + __expf(-g)) * u;
+    float g = __uint_as_float(r[2 * j]), u = __uint_as_float(r[2 * j + 1]);
+    if (act == NB_ACT_CLAMPED_GLU_PAIRS) {
+      g = fminf(g, limit);
+      u = fminf(fmaxf(u, -limit), limit) + 1.0f;
+      o[j] = g / (1.0f + __expf(-alpha * g)) * u;
+    } else {
+      o[j] = g / (1.0f + __expf(-g)) * u;
+    }
   }
   if (y_dtype == NB_BF16) {
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(y) + at;
@@ -88,8 +96,8 @@ __device__ __forceinline__ void store_swiglu_pairs(const uint32_t (&r)[16], void
 // Two accumulator buffers in tensor memory let the epilogue of one tile overlap the MMAs of the next.
 __global__ void __launch_bounds__(192, 1)
 gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w, void* __restrict__ y,
-                 int y_dtype, int ldy, const float* __restrict__ bias, int act, int M, int N, int K, int BN, int m_tiles, int n_tiles,
-                 int f16, int pair, int* status) {
+                 int y_dtype, int ldy, const float* __restrict__ bias, int act, float alpha, float limit, int M, int N, int K, int BN,
+                 int m_tiles, int n_tiles, int f16, int pair, int* status) {
   using Cfg = GemmCfg;
   const int S = Cfg::stages(BN);
   const int b_bytes = BN * kBK * 2;   // multiple of 1024 because BN is a multiple of 16
@@ -203,8 +211,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
           for (int j = 0; j < 16; ++j)
             if (n + j < N) r[j] = __float_as_uint(__uint_as_float(r[j]) + __ldg(bias + n + j));
         }
-        if (act == NB_ACT_SWIGLU_PAIRS) {  // columns 2i (gate) and 2i + 1 (up) -> output column i
-          if (m < M && n < N) store_swiglu_pairs(r, y, y_dtype, (size_t)m * ldy + (n >> 1), min(8, (N - n) >> 1));
+        if (act != NB_ACT_NONE) {  // columns 2i (gate) and 2i + 1 (up) -> output column i
+          if (m < M && n < N) store_glu_pairs(r, act, alpha, limit, y, y_dtype, (size_t)m * ldy + (n >> 1), min(8, (N - n) >> 1));
           continue;
         }
         if (pair) {
@@ -277,8 +285,8 @@ static int pick_bn(int M, int N, int sms) {
   return best;
 }
 
-static int launch_gemm(const CUtensorMap& mx, const CUtensorMap& mw, void* y, int y_dtype, int ldy, const float* bias, int act, int M,
-                       int N, int K, int bn, int f16, int pair, int* status, cudaStream_t st) {
+static int launch_gemm(const CUtensorMap& mx, const CUtensorMap& mw, void* y, int y_dtype, int ldy, const float* bias, int act, float alpha,
+                       float limit, int M, int N, int K, int bn, int f16, int pair, int* status, cudaStream_t st) {
   static bool attr_done[64] = {false};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -289,7 +297,8 @@ static int launch_gemm(const CUtensorMap& mx, const CUtensorMap& mw, void* y, in
   }
   const int m_tiles = (M + kBM - 1) / kBM, n_tiles = (N + bn - 1) / bn;
   const int grid = std::min(sm_count(), m_tiles * n_tiles);
-  gemm_bf16_kernel<<<grid, 192, GemmCfg::kSmem, st>>>(mx, mw, y, y_dtype, ldy, bias, act, M, N, K, bn, m_tiles, n_tiles, f16, pair, status);
+  gemm_bf16_kernel<<<grid, 192, GemmCfg::kSmem, st>>>(mx, mw, y, y_dtype, ldy, bias, act, alpha, limit, M, N, K, bn, m_tiles, n_tiles, f16,
+                                                         pair, status);
   return check_launch();
 }
 
@@ -334,26 +343,26 @@ static int gemm_16bit(const void* x, const void* w, int f16, int M, int N, int K
   if (int rc = make_map(&mx, x, M, K, kBM)) return rc;
   if (int rc = make_map(&mw, w, N, K, bn)) return rc;
   cudaStream_t st = (cudaStream_t)stream;
-  return launch_gemm(mx, mw, y, y_dtype, N, nullptr, NB_ACT_NONE, M, N, K, bn, f16, pair, status, st);
+  return launch_gemm(mx, mw, y, y_dtype, N, nullptr, NB_ACT_NONE, 0.f, 0.f, M, N, K, bn, f16, pair, status, st);
 }
 
 extern "C" int nb_gemm_bf16(const void* x, const void* w, int M, int N, int K, void* y, int y_dtype, int* status, void* stream) {
   return gemm_16bit(x, w, 0, M, N, K, y, y_dtype, status, stream);
 }
 
-extern "C" int nb_linear_bf16(const void* x, int ldx, const void* w, int ldw, const float* bias, int act, int M, int N, int K, void* y,
-                              int y_dtype, int ldy, int* status, void* stream) {
+extern "C" int nb_linear_bf16(const void* x, int ldx, const void* w, int ldw, const float* bias, int act, float alpha, float limit, int M,
+                              int N, int K, void* y, int y_dtype, int ldy, int* status, void* stream) {
   if (!x || !w || !y || M < 1 || N < 1 || K < 1 || ldx < K || ldw < K) return NB_ERR_ARG;
-  if ((y_dtype != NB_BF16 && y_dtype != NB_F32) || (act != NB_ACT_NONE && act != NB_ACT_SWIGLU_PAIRS)) return NB_ERR_ARG;
-  if (act == NB_ACT_SWIGLU_PAIRS && N % 2) return NB_ERR_SHAPE;
-  if (ldy < (act == NB_ACT_SWIGLU_PAIRS ? N / 2 : N)) return NB_ERR_ARG;
+  if ((y_dtype != NB_BF16 && y_dtype != NB_F32) || act < NB_ACT_NONE || act > NB_ACT_CLAMPED_GLU_PAIRS) return NB_ERR_ARG;
+  if (act != NB_ACT_NONE && N % 2) return NB_ERR_SHAPE;
+  if (ldy < (act != NB_ACT_NONE ? N / 2 : N)) return NB_ERR_ARG;
   if ((uintptr_t)x % 16 || (uintptr_t)w % 16 || ldx % 8 || ldw % 8 || (uintptr_t)y % 4) return NB_ERR_ALIGN;
   if (int rc = check_device()) return rc;
   const int bn = N < 128 ? (N + 15) / 16 * 16 : pick_bn(M, N, sm_count());
   CUtensorMap mx, mw;
   if (int rc = make_map(&mx, x, M, K, kBM, ldx)) return rc;
   if (int rc = make_map(&mw, w, N, K, bn, ldw)) return rc;
-  return launch_gemm(mx, mw, y, y_dtype, ldy, bias, act, M, N, K, bn, 0, 0, status, (cudaStream_t)stream);
+  return launch_gemm(mx, mw, y, y_dtype, ldy, bias, act, alpha, limit, M, N, K, bn, 0, 0, status, (cudaStream_t)stream);
 }
 
 extern "C" int nb_gemm_prefill(const void* x, int x_dtype, int M, const uint8_t* packed, const void* codebook, int cb_dtype, int bits,

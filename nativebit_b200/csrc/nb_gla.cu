@@ -1,5 +1,6 @@
 // Gated linear attention: per head a (dim x vdim) state S, S <- diag(alpha) S + k v^T, o = S^T q, with a decay alpha per
-// key channel from a low-rank projection.
+// key channel: from a low-rank projection beside a projected key (NB_GLA_LOW_RANK), or a forget gate above a lower bound
+// with the key 1 - alpha (NB_GLA_FORGET, the HGRN2 recurrence).
 //
 // Prompts run in chunks of 64 tokens (the chunkwise form of "Gated Linear Attention Transformers with Hardware-Efficient
 // Training", Yang, Wang, Shen, Panda and Kim): every chunk's contribution to the state in parallel, a scan over the chunks,
@@ -30,8 +31,42 @@ struct GlaWs {
 
 __host__ __device__ inline int gla_chunks(int T) { return (T + kGC - 1) / kGC; }
 
+// ---- the forget gate: alpha = 1 - om * sigmoid(-z) with om = 1 - lower; the key is om * sigmoid(-z), without the
+// cancellation of 1 - alpha.
+__device__ __forceinline__ float forget_key(float z, float om) { return om * sigmoid_f(-z); }
+__device__ __forceinline__ float forget_key_fast(float z, float om) { return __fdividef(om, 1.f + __expf(z)); }
+// log alpha; a gate that closes completely counts as the smallest normal number
+__device__ __forceinline__ float forget_log(float z, float lower) {
+  const float om = 1.f - lower, k = forget_key(z, om);
+  return k < 0.5f ? log1pf(-k) : logf(fmaxf(lower + om * sigmoid_f(z), 1.17549435e-38f));
+}
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+// q and k as the recurrence takes them, from what the projection left (fp32 functions): `ch` counts all heads' channels.
+template <int kKind> __device__ __forceinline__ float gla_q(float q, float scale) { return kKind == NB_GLA_FORGET ? silu_f(q) : q * scale; }
+template <int kKind> __device__ __forceinline__ float gla_k(const nb_gla_args& p, float k, int ch) {
+  return kKind == NB_GLA_FORGET ? forget_key(k + p.a2_b[ch], 1.f - p.lower[ch]) : k;
+}
+
 // ---- decays.  grid (sub-blocks, channel tiles, B); a thread owns one channel of 16 tokens.
 constexpr int kDecThreads = 128;
+template <typename T> __global__ void __launch_bounds__(kDecThreads) gla_forget_kernel(const nb_gla_args p, GlaWs w) {
+  const int t0 = blockIdx.x * kGS, b = blockIdx.z, ch = blockIdx.y * kDecThreads + threadIdx.x, HD = p.H * p.dim;
+  if (ch >= HD) return;
+  const int cnt = min(kGS, p.T - t0);
+  const T* z = reinterpret_cast<const T*>(p.p) + (size_t)(b * p.T + t0) * p.ldp + p.k_off + ch;
+  float* out = w.bl + (size_t)(b * p.T + t0) * HD + ch;
+  const float bias = p.a2_b[ch], lower = p.lower[ch];
+  float v[kGS], sum = 0.f;
+#pragma unroll
+  for (int t = 0; t < kGS; ++t) v[t] = t < cnt ? to_f(z[(size_t)t * p.ldp]) : 0.f;
+#pragma unroll
+  for (int t = 0; t < kGS; ++t) {
+    sum += forget_log(v[t] + bias, lower);
+    if (t < cnt) out[(size_t)t * HD] = sum;
+  }
+}
+
 template <typename T> __global__ void __launch_bounds__(kDecThreads) gla_decay_kernel(const nb_gla_args p, GlaWs w) {
   extern __shared__ __align__(16) float as[];           // [kGS][a_rank]
   const int t0 = blockIdx.x * kGS, b = blockIdx.z, ch = blockIdx.y * kDecThreads + threadIdx.x, HD = p.H * p.dim;
@@ -66,7 +101,7 @@ template <typename T> __global__ void __launch_bounds__(kDecThreads) gla_decay_k
 
 // ---- what a chunk adds to the state: U[d][v] = sum_t k_t[d] exp(decay from t to the chunk's end) v_t[v].
 // grid (chunks, H * d tiles * v tiles, B), 64 x 64 outputs per CTA.
-template <typename T> __global__ void __launch_bounds__(256) gla_state_kernel(const nb_gla_args p, GlaWs w, int dtiles, int vtiles) {
+template <typename T, int kKind> __global__ void __launch_bounds__(256) gla_state_kernel(const nb_gla_args p, GlaWs w, int dtiles, int vtiles) {
   __shared__ __align__(16) float ks[kGC][64 + 4], vs[kGC][64 + 4];
   __shared__ float tot[kGSubs][64];                     // log decay of a whole sub-block
   const int n = blockIdx.x, b = blockIdx.z, tid = threadIdx.x;
@@ -86,7 +121,7 @@ template <typename T> __global__ void __launch_bounds__(256) gla_state_kernel(co
     if (t < cnt && d < p.dim) {
       float e = tot[s][c] - bl[(size_t)t * HD + d];
       for (int m = s + 1; m < kGSubs; ++m) e += tot[m][c];
-      kv = to_f(base[(size_t)t * p.ldp + p.k_off + h * p.dim + d]) * expf(e);
+      kv = gla_k<kKind>(p, to_f(base[(size_t)t * p.ldp + p.k_off + h * p.dim + d]), h * p.dim + d) * expf(e);
     }
     ks[t][c] = kv;
     vs[t][c] = (t < cnt && v < p.vdim) ? to_f(base[(size_t)t * p.ldp + p.v_off + h * p.vdim + v]) : 0.f;
@@ -147,7 +182,7 @@ __global__ void __launch_bounds__(256) gla_scan_kernel(const nb_gla_args p, GlaW
 // A[t][s] = sum_d q_t[d] k_s[d] exp(decay from s to t).  grid (chunks, H, B).  A is built 4 x 4 per thread; for tokens of
 // different sub-blocks the decay is split at the start of t's sub-block, inside a sub-block at the start of t's group of
 // four, and inside a group of four it is taken pair by pair.
-template <typename T> __global__ void __launch_bounds__(256) gla_output_kernel(const nb_gla_args p, GlaWs w) {
+template <typename T, int kKind> __global__ void __launch_bounds__(256) gla_output_kernel(const nb_gla_args p, GlaWs w) {
   extern __shared__ __align__(16) float gsm[];
   constexpr int ld = 64 + 4;
   float* as = gsm;                      // [64][ld]  A, transposed: as[s][t]
@@ -166,7 +201,7 @@ template <typename T> __global__ void __launch_bounds__(256) gla_output_kernel(c
     for (int i = tid; i < kGC * 64; i += 256) {
       const int t = i >> 6, c = i & 63, d = d0 + c;
       const bool in = t < cnt && d < p.dim;
-      qt[c * ld + t] = in ? to_f(base[(size_t)t * p.ldp + p.q_off + h * p.dim + d]) * qscale : 0.f;
+      qt[c * ld + t] = in ? gla_q<kKind>(to_f(base[(size_t)t * p.ldp + p.q_off + h * p.dim + d]), qscale) : 0.f;
       bt[c * ld + t] = in ? bl[(size_t)t * HD + d] : 0.f;
     }
     for (int i = tid; i < kGSubs * 64; i += 256) {
@@ -181,7 +216,7 @@ template <typename T> __global__ void __launch_bounds__(256) gla_output_kernel(c
     load_tile(d0);
     for (int i = tid; i < kGC * 64; i += 256) {
       const int t = i >> 6, c = i & 63, d = d0 + c;
-      kt[c * ld + t] = (t < cnt && d < p.dim) ? to_f(base[(size_t)t * p.ldp + p.k_off + h * p.dim + d]) : 0.f;
+      kt[c * ld + t] = (t < cnt && d < p.dim) ? gla_k<kKind>(p, to_f(base[(size_t)t * p.ldp + p.k_off + h * p.dim + d]), h * p.dim + d) : 0.f;
     }
     __syncthreads();
     const int dn = min(64, p.dim - d0);
@@ -274,7 +309,7 @@ template <typename T> __global__ void __launch_bounds__(256) gla_output_kernel(c
   }
 }
 
-// ---- out = RMSNorm(o) * norm_w * silu(g), one warp per (row, head)
+// ---- out = RMSNorm(o) * norm_w * silu(g) (no gate with g_off < 0), one warp per (row, head)
 template <typename T> __global__ void __launch_bounds__(256) gla_finish_kernel(const nb_gla_args p, GlaWs w) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const size_t rh = (size_t)blockIdx.x * 8 + warp;
@@ -287,7 +322,7 @@ template <typename T> __global__ void __launch_bounds__(256) gla_finish_kernel(c
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.vdim + p.eps);
   const T* g = reinterpret_cast<const T*>(p.p) + row * p.ldp + p.g_off + h * p.vdim;
   T* out = reinterpret_cast<T*>(p.out) + row * p.ldo + h * p.vdim;
-  for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * inv * p.norm_w[i] * silu_f(to_f(g[i])));
+  for (int i = lane; i < p.vdim; i += 32) out[i] = from_f<T>(o[i] * inv * p.norm_w[i] * (p.g_off < 0 ? 1.f : silu_f(to_f(g[i]))));
 }
 
 // ---- the same two kernels for bf16 projections on the tensor cores.  q, k and v are bf16 as they are; everything the
@@ -356,8 +391,23 @@ __device__ __forceinline__ bool sub_block_totals(float* tot, const float* bl, in
   return deep;
 }
 
+// Bias and 1 - lower bound of two neighbouring channels, and the keys of the pair.
+struct ForgetPair {
+  float2 bias, om;
+  __device__ ForgetPair(const nb_gla_args& p, int kind, int ch, int d, int dn) {
+    bias = om = make_float2(0.f, 0.f);
+    if (kind != NB_GLA_FORGET) return;
+    if (d < dn) { bias.x = p.a2_b[ch]; om.x = 1.f - p.lower[ch]; }
+    if (d + 1 < dn) { bias.y = p.a2_b[ch + 1]; om.y = 1.f - p.lower[ch + 1]; }
+  }
+  template <int kKind> __device__ __forceinline__ float2 key(uint32_t kk) const {
+    if (kKind != NB_GLA_FORGET) return make_float2(bf_lo(kk), bf_hi(kk));
+    return make_float2(forget_key_fast(bf_lo(kk) + bias.x, om.x), forget_key_fast(bf_hi(kk) + bias.y, om.y));
+  }
+};
+
 // grid (chunks, H * d tiles, B): 64 channels x vdim of a chunk's contribution.
-template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_kernel(const nb_gla_args p, GlaWs w, int dtiles, int vec) {
+template <int VD, int kKind> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_kernel(const nb_gla_args p, GlaWs w, int dtiles, int vec) {
   extern __shared__ __align__(16) uint8_t gsm_raw[];
   GlaStateSmem<VD>& sm = *reinterpret_cast<GlaStateSmem<VD>*>(gsm_raw);
   const int n = blockIdx.x, h = blockIdx.y / dtiles, d0 = (blockIdx.y - h * dtiles) * 64, b = blockIdx.z;
@@ -369,6 +419,7 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_ke
   stage_decays(sm.bl, bl, HD, dn, cnt, vec);
   stage_rows(sm.k, kGmLd, base + p.k_off + h * p.dim + d0, p.ldp, 64, dn, cnt, vec);
   stage_rows(sm.v, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  const ForgetPair fp(p, kKind, h * p.dim + d0 + 2 * lane, 2 * lane, dn);   // of this thread's pair of channels below
   stage_wait();
   __syncthreads();
   sub_block_totals(sm.tot, sm.bl, cnt);
@@ -383,7 +434,8 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_state_mma_ke
     for (int m = 1; m < kGSubs; ++m)
       if (m > s) { ex += sm.tot[m * 64 + d]; ey += sm.tot[m * 64 + d + 1]; }
     uint32_t hi, lo;
-    split_bf16(bf_lo(kk) * __expf(ex), bf_hi(kk) * __expf(ey), hi, lo);
+    const float2 key = fp.key<kKind>(kk);
+    split_bf16(key.x * __expf(ex), key.y * __expf(ey), hi, lo);
     if (t >= cnt) hi = lo = 0u;
     *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
     *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
@@ -440,7 +492,7 @@ template <int VD> struct GlaOutSmem {
 // at the chunk's start; then the scores against the values, the norm over the head's outputs and the gate.
 //   q . k over sub-blocks i > j: (q exp(bl)) . (k exp(tot_j - bl)) * exp(tot_{j+1} + .. + tot_{i-1}), the last on q's side;
 //   i == j: the same with exp(-tot_i), as long as no channel of the tile decays past kSplitLimit inside the sub-block.
-template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_kernel(const nb_gla_args p, GlaWs w, int vec) {
+template <int VD, int kKind> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_kernel(const nb_gla_args p, GlaWs w, int vec) {
   extern __shared__ __align__(16) uint8_t gsm_raw[];
   GlaOutSmem<VD>& sm = *reinterpret_cast<GlaOutSmem<VD>*>(gsm_raw);
   const int n = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -498,12 +550,14 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
       f[8 * 64] = deep ? 0.f : __expf(-a2);
       f[9 * 64] = deep ? 0.f : __expf(-a3);
     }
+    const ForgetPair fp(p, kKind, h * p.dim + d0 + 2 * lane, 2 * lane, dn);
     for (int i = tid; i < kGC * 32; i += kGmThreads) {
       const int t = i >> 5, d = (i & 31) * 2;
       const uint32_t kk = *reinterpret_cast<const uint32_t*>(sm.k + t * kGmLd + d);
       const float* tt = sm.tot + (t / kGS) * 64 + d;
       uint32_t hi, lo;
-      split_bf16(bf_lo(kk) * __expf(tt[0] - sm.bl[t * kGbLd + d]), bf_hi(kk) * __expf(tt[1] - sm.bl[t * kGbLd + d + 1]), hi, lo);
+      const float2 key = fp.key<kKind>(kk);
+      split_bf16(key.x * __expf(tt[0] - sm.bl[t * kGbLd + d]), key.y * __expf(tt[1] - sm.bl[t * kGbLd + d + 1]), hi, lo);
       if (t >= cnt) hi = lo = 0u;
       *reinterpret_cast<uint32_t*>(sm.khi + t * kGmLd + d) = hi;
       *reinterpret_cast<uint32_t*>(sm.klo + t * kGmLd + d) = lo;
@@ -518,8 +572,8 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
       for (int j = 0; j < 4; ++j) {
         const int r = (j & 1) ? rb : ra, c = kk + c2 + (j >> 1) * 8;
         const uint32_t qq = *reinterpret_cast<const uint32_t*>(sm.q + r * kGmLd + c);
-        qd[j][0] = bf_lo(qq) * qscale * __expf(sm.bl[r * kGbLd + c]);
-        qd[j][1] = bf_hi(qq) * qscale * __expf(sm.bl[r * kGbLd + c + 1]);
+        qd[j][0] = (kKind == NB_GLA_FORGET ? silu_fast(bf_lo(qq)) : bf_lo(qq) * qscale) * __expf(sm.bl[r * kGbLd + c]);
+        qd[j][1] = (kKind == NB_GLA_FORGET ? silu_fast(bf_hi(qq)) : bf_hi(qq) * qscale) * __expf(sm.bl[r * kGbLd + c + 1]);
       }
       auto fragment = [&](const float* f, uint32_t (&hi)[4], uint32_t (&lo)[4]) {   // f: per-channel factor or null
 #pragma unroll
@@ -582,8 +636,9 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
             if (s > t || t >= cnt) continue;
             float sum = 0.f;
             for (int d = 0; d < dn; ++d)
-              sum += to_f(sm.q[t * kGmLd + d]) * __expf(sm.bl[t * kGbLd + d] - sm.bl[s * kGbLd + d]) * to_f(sm.k[s * kGmLd + d]);
-            sc[j][x][e] += sum * qscale;
+              sum += gla_q<kKind>(to_f(sm.q[t * kGmLd + d]), qscale) * __expf(sm.bl[t * kGbLd + d] - sm.bl[s * kGbLd + d]) *
+                     gla_k<kKind>(p, to_f(sm.k[s * kGmLd + d]), h * p.dim + d0 + d);
+            sc[j][x][e] += sum;
           }
       }
     }
@@ -591,7 +646,8 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
   __syncthreads();
   // the values, the gate and the norm's weights take the place of the state and the factors
   stage_rows(sm.shi, VD + 8, base + p.v_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
-  stage_rows(sm.slo, VD + 8, base + p.g_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
+  const bool gated = p.g_off >= 0;
+  if (gated) stage_rows(sm.slo, VD + 8, base + p.g_off + h * p.vdim, p.ldp, VD, p.vdim, cnt, vec);
   for (int i = tid; i < VD; i += kGmThreads) sm.fac[i] = i < p.vdim ? p.norm_w[i] : 0.f;
   stage_wait();
   __syncthreads();
@@ -640,8 +696,8 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
       const uint32_t gg = *reinterpret_cast<const uint32_t*>(g + v);
       const float2 nw = *reinterpret_cast<const float2*>(sm.fac + v);
       const float gx = bf_lo(gg), gy = bf_hi(gg);
-      const float x = o[i][2 * half] * inv * nw.x * __fdividef(gx, 1.f + __expf(-gx));
-      const float y = o[i][2 * half + 1] * inv * nw.y * __fdividef(gy, 1.f + __expf(-gy));
+      const float x = o[i][2 * half] * inv * nw.x * (gated ? __fdividef(gx, 1.f + __expf(-gx)) : 1.f);
+      const float y = o[i][2 * half + 1] * inv * nw.y * (gated ? __fdividef(gy, 1.f + __expf(-gy)) : 1.f);
       if (vec) {
         if (v < p.vdim) *reinterpret_cast<uint32_t*>(out + v) = pack_bf16(x, y);
       } else {
@@ -659,7 +715,7 @@ template <int VD> __global__ void __launch_bounds__(kGmThreads) gla_output_mma_k
 constexpr int kGdThreads = 256, kGdWarps = kGdThreads / 32;
 constexpr int kGdPre = 8;              // rows of the state (four columns each) a thread may hold ahead of the wait
 
-__global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_args p) {
+template <int kKind> __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_args p) {
   extern __shared__ __align__(16) float gdm[];
   __shared__ float red[kGdWarps], ssq;
   cg::cluster_group cluster = cg::this_cluster();
@@ -680,7 +736,7 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_arg
     const int d = g0 + i * groups0;
     sreg[i] = (pre && g0 < groups0 && d < p.dim) ? st[(size_t)d * quads + c0 + cc0] : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  const bool short_rank = p.lda2 <= 16 && p.dim <= kGdThreads;   // a row of W_a2 is one or two 16-byte loads
+  const bool short_rank = kKind == NB_GLA_LOW_RANK && p.lda2 <= 16 && p.dim <= kGdThreads;   // a row of W_a2 is one or two 16-byte loads
   const bf16* w2 = reinterpret_cast<const bf16*>(p.a2) + (size_t)(h * p.dim) * p.lda2;
   uint4 wa = make_uint4(0u, 0u, 0u, 0u), wb = wa;
   float bias = 0.f;
@@ -689,6 +745,8 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_arg
     if (p.lda2 > 8) wb = *reinterpret_cast<const uint4*>(w2 + (size_t)tid * p.lda2 + 8);
     bias = p.a2_b[h * p.dim + tid];
   }
+  float lower = 0.f;
+  if (kKind == NB_GLA_FORGET && tid < p.dim) { bias = p.a2_b[h * p.dim + tid]; lower = p.lower[h * p.dim + tid]; }
   pdl_enter();
   const float* row = reinterpret_cast<const float*>(p.p) + (size_t)b * p.ldp;
   const float* vrow = row + p.v_off + h * p.vdim;
@@ -701,6 +759,13 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_arg
   for (int d = tid; d < p.dim; d += kGdThreads) {
     const int ch = h * p.dim + d;
     const float k = row[p.k_off + ch], q = row[p.q_off + ch];
+    if constexpr (kKind == NB_GLA_FORGET) {
+      const float lo = d == tid ? lower : p.lower[ch], zf = k + (d == tid ? bias : p.a2_b[ch]), om = 1.f - lo;
+      al[d] = lo + om * sigmoid_f(zf);
+      ks[d] = forget_key(zf, om);
+      qs[d] = silu_f(q);
+      continue;
+    }
     float z;
     if (short_rank) {
       z = bias;
@@ -766,16 +831,21 @@ __global__ void __launch_bounds__(kGdThreads) gla_decode_kernel(const nb_gla_arg
   for (int i = tid; i < 4 * cn; i += kGdThreads) {
     const int v = 4 * c0 + i;
     if (v < p.vdim)
-      reinterpret_cast<float*>(p.out)[(size_t)b * p.ldo + h * p.vdim + v] = os[i] * inv * p.norm_w[v] * silu_f(row[p.g_off + h * p.vdim + v]);
+      reinterpret_cast<float*>(p.out)[(size_t)b * p.ldo + h * p.vdim + v] = os[i] * inv * p.norm_w[v] * (p.g_off < 0 ? 1.f : silu_f(row[p.g_off + h * p.vdim + v]));
   }
 }
 
-template <typename T> static int gla_prefill(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
-  const int chunks = gla_chunks(a.T), subs = (a.T + kGS - 1) / kGS, dt = (a.dim + 63) / 64, vt = (a.vdim + 63) / 64;
-  const int HD = a.H * a.dim;
-  gla_decay_kernel<T><<<dim3(subs, (HD + kDecThreads - 1) / kDecThreads, a.B), kDecThreads, (size_t)kGS * a.a_rank * 4, st>>>(a, w);
-  if (int rc = check_launch()) return rc;
-  gla_state_kernel<T><<<dim3(chunks, a.H * dt * vt, a.B), 256, 0, st>>>(a, w, dt, vt);
+template <typename T, int kKind> static int launch_decays(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
+  const dim3 grid((a.T + kGS - 1) / kGS, (a.H * a.dim + kDecThreads - 1) / kDecThreads, a.B);
+  if (kKind == NB_GLA_FORGET) gla_forget_kernel<T><<<grid, kDecThreads, 0, st>>>(a, w);
+  else gla_decay_kernel<T><<<grid, kDecThreads, (size_t)kGS * a.a_rank * 4, st>>>(a, w);
+  return check_launch();
+}
+
+template <typename T, int kKind> static int gla_prefill(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
+  const int chunks = gla_chunks(a.T), dt = (a.dim + 63) / 64, vt = (a.vdim + 63) / 64;
+  if (int rc = launch_decays<T, kKind>(a, w, st)) return rc;
+  gla_state_kernel<T, kKind><<<dim3(chunks, a.H * dt * vt, a.B), 256, 0, st>>>(a, w, dt, vt);
   if (int rc = check_launch()) return rc;
   gla_scan_kernel<<<dim3((a.dim * (a.lds / 4) + 255) / 256, a.B * a.H), 256, 0, st>>>(a, w, chunks);
   if (int rc = check_launch()) return rc;
@@ -784,10 +854,10 @@ template <typename T> static int gla_prefill(const nb_gla_args& a, const GlaWs& 
   int dev = 0;
   cudaGetDevice(&dev);
   if (!done[dev & 63]) {
-    if (cudaError_t e = cudaFuncSetAttribute(gla_output_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return record_cuda_error(e);
+    if (cudaError_t e = cudaFuncSetAttribute(gla_output_kernel<T, kKind>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)) return record_cuda_error(e);
     done[dev & 63] = true;
   }
-  gla_output_kernel<T><<<dim3(chunks, a.H, a.B), 256, smem, st>>>(a, w);
+  gla_output_kernel<T, kKind><<<dim3(chunks, a.H, a.B), 256, smem, st>>>(a, w);
   if (int rc = check_launch()) return rc;
   const size_t rh = (size_t)a.B * a.T * a.H;
   gla_finish_kernel<T><<<(unsigned)((rh + 7) / 8), 256, 0, st>>>(a, w);
@@ -795,41 +865,50 @@ template <typename T> static int gla_prefill(const nb_gla_args& a, const GlaWs& 
 }
 
 // bf16 projections with vdim <= VD: decay, state, scan and output kernels, the last with the norm and the gate.
-template <int VD> static int gla_prefill_mma(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
-  const int chunks = gla_chunks(a.T), subs = (a.T + kGS - 1) / kGS, dt = (a.dim + 63) / 64, HD = a.H * a.dim;
+template <int VD, int kKind> static int gla_prefill_mma(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
+  const int chunks = gla_chunks(a.T), dt = (a.dim + 63) / 64;
   const int vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ldp % 8 == 0 && a.q_off % 8 == 0 && a.k_off % 8 == 0 && a.v_off % 8 == 0 &&
-                  a.g_off % 8 == 0 && a.ldo % 2 == 0 && (uintptr_t)a.p % 16 == 0 && (uintptr_t)a.out % 4 == 0;
+                  (a.g_off < 0 || a.g_off % 8 == 0) && a.ldo % 2 == 0 && (uintptr_t)a.p % 16 == 0 && (uintptr_t)a.out % 4 == 0;
   static bool done[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!done[dev & 63]) {
-    if (cudaError_t e = cudaFuncSetAttribute(gla_state_mma_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaStateSmem<VD>)))
+    if (cudaError_t e = cudaFuncSetAttribute(gla_state_mma_kernel<VD, kKind>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaStateSmem<VD>)))
       return record_cuda_error(e);
-    if (cudaError_t e = cudaFuncSetAttribute(gla_output_mma_kernel<VD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaOutSmem<VD>)))
+    if (cudaError_t e = cudaFuncSetAttribute(gla_output_mma_kernel<VD, kKind>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)sizeof(GlaOutSmem<VD>)))
       return record_cuda_error(e);
     done[dev & 63] = true;
   }
-  gla_decay_kernel<bf16><<<dim3(subs, (HD + kDecThreads - 1) / kDecThreads, a.B), kDecThreads, (size_t)kGS * a.a_rank * 4, st>>>(a, w);
-  if (int rc = check_launch()) return rc;
-  gla_state_mma_kernel<VD><<<dim3(chunks, a.H * dt, a.B), kGmThreads, sizeof(GlaStateSmem<VD>), st>>>(a, w, dt, vec);
+  if (int rc = launch_decays<bf16, kKind>(a, w, st)) return rc;
+  gla_state_mma_kernel<VD, kKind><<<dim3(chunks, a.H * dt, a.B), kGmThreads, sizeof(GlaStateSmem<VD>), st>>>(a, w, dt, vec);
   if (int rc = check_launch()) return rc;
   gla_scan_kernel<<<dim3((a.dim * (a.lds / 4) + 255) / 256, a.B * a.H), 256, 0, st>>>(a, w, chunks);
   if (int rc = check_launch()) return rc;
-  gla_output_mma_kernel<VD><<<dim3(chunks, a.H, a.B), kGmThreads, sizeof(GlaOutSmem<VD>), st>>>(a, w, vec);
+  gla_output_mma_kernel<VD, kKind><<<dim3(chunks, a.H, a.B), kGmThreads, sizeof(GlaOutSmem<VD>), st>>>(a, w, vec);
   return check_launch();
 }
 
+template <int kKind> static int gla_prefill_kind(const nb_gla_args& a, const GlaWs& w, cudaStream_t st) {
+  if (a.dtype == NB_F32) return gla_prefill<float, kKind>(a, w, st);
+  return a.vdim <= 64    ? gla_prefill_mma<64, kKind>(a, w, st)
+         : a.vdim <= 128 ? gla_prefill_mma<128, kKind>(a, w, st)
+         : a.vdim <= 256 ? gla_prefill_mma<256, kKind>(a, w, st)
+                         : gla_prefill<bf16, kKind>(a, w, st);
+}
+
 static int gla_check(const nb_gla_args* a) {
-  if (!a || !a->p || !a->out || !a->state || !a->a2 || !a->a2_b || !a->norm_w || a->B < 1 || a->T < 1 || a->H < 1 || a->dim < 1 || a->vdim < 1 ||
-      a->a_rank < 1 || !(a->tau > 0.f))
+  if (!a || !a->p || !a->out || !a->state || !a->a2_b || !a->norm_w || a->B < 1 || a->T < 1 || a->H < 1 || a->dim < 1 || a->vdim < 1)
     return NB_ERR_ARG;
+  const bool low_rank = a->kind == NB_GLA_LOW_RANK;
+  if (low_rank ? !a->a2 || a->a_rank < 1 || !(a->tau > 0.f) : a->kind != NB_GLA_FORGET || !a->lower) return NB_ERR_ARG;
   if (a->dtype != NB_BF16 && a->dtype != NB_F32) return NB_ERR_ARG;
   const int hd = a->H * a->dim, hv = a->H * a->vdim;
-  if (a->q_off < 0 || a->k_off < 0 || a->v_off < 0 || a->g_off < 0 || a->a_off < 0 || a->q_off + hd > a->ldp || a->k_off + hd > a->ldp ||
-      a->v_off + hv > a->ldp || a->g_off + hv > a->ldp || a->a_off + a->a_rank > a->ldp || a->lda2 < a->a_rank || a->ldo < hv ||
+  if (a->q_off < 0 || a->k_off < 0 || a->v_off < 0 || (low_rank && (a->g_off < 0 || a->a_off < 0)) || a->q_off + hd > a->ldp ||
+      a->k_off + hd > a->ldp || a->v_off + hv > a->ldp || (a->g_off >= 0 && a->g_off + hv > a->ldp) ||
+      (low_rank && (a->a_off + a->a_rank > a->ldp || a->lda2 < a->a_rank)) || a->ldo < hv ||
       a->lds < a->vdim || a->lds % 4 || a->H > 65535 || a->B > 65535 || (long long)a->B * a->H > 65535)
     return NB_ERR_SHAPE;
-  if ((uintptr_t)a->state % 16 || (uintptr_t)a->a2 % 16 || a->lda2 % 8) return NB_ERR_ALIGN;
+  if ((uintptr_t)a->state % 16 || (low_rank && ((uintptr_t)a->a2 % 16 || a->lda2 % 8))) return NB_ERR_ALIGN;
   return NB_OK;
 }
 
@@ -851,7 +930,7 @@ extern "C" int nb_gla_prefill(const nb_gla_args* a, void* workspace, size_t work
   if (!workspace || workspace_bytes < nb_gla_workspace_bytes(a->B, a->T, a->H, a->dim, a->vdim)) return NB_ERR_WORKSPACE;
   if ((uintptr_t)workspace % 256) return NB_ERR_ALIGN;
   const int dt = (a->dim + 63) / 64, vt = (a->vdim + 63) / 64;
-  if ((long long)a->H * dt * vt > 65535 || (size_t)kGS * a->a_rank * 4 > 48 * 1024 || (a->H * a->dim + kDecThreads - 1) / kDecThreads > 65535)
+  if ((long long)a->H * dt * vt > 65535 || (a->kind == NB_GLA_LOW_RANK && (size_t)kGS * a->a_rank * 4 > 48 * 1024) || (a->H * a->dim + kDecThreads - 1) / kDecThreads > 65535)
     return NB_ERR_SHAPE;
   if (int rc = check_device()) return rc;
   const size_t rows = (size_t)a->B * a->T, ch = (size_t)a->B * gla_chunks(a->T) * a->H;
@@ -865,11 +944,7 @@ extern "C" int nb_gla_prefill(const nb_gla_args* a, void* workspace, size_t work
   base += round256(ch * a->dim * 4);
   w.o = reinterpret_cast<float*>(base);
   cudaStream_t st = (cudaStream_t)stream;
-  if (a->dtype == NB_F32) return gla_prefill<float>(*a, w, st);
-  return a->vdim <= 64    ? gla_prefill_mma<64>(*a, w, st)
-         : a->vdim <= 128 ? gla_prefill_mma<128>(*a, w, st)
-         : a->vdim <= 256 ? gla_prefill_mma<256>(*a, w, st)
-                          : gla_prefill<bf16>(*a, w, st);
+  return a->kind == NB_GLA_FORGET ? gla_prefill_kind<NB_GLA_FORGET>(*a, w, st) : gla_prefill_kind<NB_GLA_LOW_RANK>(*a, w, st);
 }
 
 extern "C" int nb_gla_decode(const nb_gla_args* a, void* stream) {
@@ -894,5 +969,5 @@ extern "C" int nb_gla_decode(const nb_gla_args* a, void* stream) {
   attr[1].val.clusterDim.z = S;
   cfg.attrs = attr;
   cfg.numAttrs = 2;
-  return record_cuda_error(cudaLaunchKernelEx(&cfg, gla_decode_kernel, *a));
+  return record_cuda_error(cudaLaunchKernelEx(&cfg, a->kind == NB_GLA_FORGET ? gla_decode_kernel<NB_GLA_FORGET> : gla_decode_kernel<NB_GLA_LOW_RANK>, *a));
 }

@@ -27,6 +27,15 @@ __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z));
 // log(sigmoid(z)) without overflow on either side
 __device__ __forceinline__ float log_sigmoid_f(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
+// Gated pair behind a product: silu(g) * u, or the clamped form.
+__device__ __forceinline__ float glu_f(int act, float alpha, float limit, float g, float u) {
+  if (act == NB_ACT_CLAMPED_GLU_PAIRS) {
+    g = fminf(g, limit);
+    return g * sigmoid_f(alpha * g) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+  }
+  return silu_f(g) * u;
+}
+
 // Sum over the block; `red` has one float per warp and is used by this call only (no barrier protects it afterwards).
 template <int kWarps> __device__ __forceinline__ float block_sum(float v, float* red) {
   v = warp_sum(v);

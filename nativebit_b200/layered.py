@@ -1,11 +1,14 @@
 """Layered decoders: models that list their layers one by one, each with its own mixer (latent attention over a
-sliding window, gated linear attention) and feed-forward or none, and norms before and after every sublayer,
+sliding window, gated linear attention, several branches side by side) and feed-forward or none, and a residual of one
+of two kinds: a norm before and after every sublayer,
 
-    x <- x + post(sublayer(pre(x))).
+    x <- x + post(sublayer(pre(x))),
 
-A model family describes its layers with the classes below (see nerulorn.py); this file runs them: `LayeredDecoder`
-takes prompts and portions of prompts through the matrix-product kernels, `LayeredSession` decodes single tokens
-through the fused matvec chain in a CUDA graph.  The activation dtype is bf16 or fp32; the residual stream, norms,
+or hyper-connections, several streams that every sublayer reads as a weighted sum and leaves mixed (`Link`).
+
+A model family describes its layers with the classes below (see nerulorn.py, nabalix.py); this file runs them:
+`LayeredDecoder` takes prompts and portions of prompts through the matrix-product kernels, `LayeredSession` decodes single
+tokens through the fused matvec chain in a CUDA graph.  The activation dtype is bf16 or fp32; the residual stream, norms,
 positions, attention scores and weights, decays and recurrent states are fp32 in both, and a single sequence's decode
 step has fp32 activations throughout (only the latent cache follows the dtype)."""
 from __future__ import annotations
@@ -69,6 +72,23 @@ class LatentCache:
     def reset(self) -> None:
         """Rows past the position are never read: nothing to clear."""
 
+    def carried(self) -> list[torch.Tensor]:
+        return []
+
+
+class KeyValueCache:
+    """Keys of a layer's key/value heads, then their values, one row per position: (B, context, row) of the activation dtype."""
+
+    def __init__(self, batch: int, context_len: int, keys: int, values: int, dtype: torch.dtype, device):
+        self.v_off = L.pad8(keys)
+        self.rows = torch.zeros(batch, context_len, self.v_off + L.pad8(values), dtype=dtype, device=device)
+
+    def reset(self) -> None:
+        """Rows past the position are never read: nothing to clear."""
+
+    def carried(self) -> list[torch.Tensor]:
+        return []
+
 
 class RecurrentState:
     """(B, heads, dim, padded vdim) fp32, carried from token to token."""
@@ -78,6 +98,24 @@ class RecurrentState:
 
     def reset(self) -> None:
         self.s.zero_()
+
+    def carried(self) -> list[torch.Tensor]:
+        """What a step changes in place."""
+        return [self.s]
+
+
+class BranchCaches:
+    """One cache or state per branch of a mixer."""
+
+    def __init__(self, parts: list):
+        self.parts = parts
+
+    def reset(self) -> None:
+        for p in self.parts:
+            p.reset()
+
+    def carried(self) -> list[torch.Tensor]:
+        return [t for p in self.parts for t in p.carried()]
 
 
 # ---------------------------------------------------------------------- pieces of a layer
@@ -133,7 +171,7 @@ class LatentAttention:
                     ldc=cache.rows.shape[2], cos2=cos_sin[0].data_ptr(), sin2=cos_sin[1].data_ptr(), scale=self.scale, window=self.window,
                     cache=cache.rows.data_ptr())
 
-    def prompt(self, h: torch.Tensor, span: Span, cache: LatentCache, cos_sin) -> torch.Tensor:
+    def prompt(self, h: torch.Tensor, span: Span, cache: LatentCache, cos_sin) -> list[torch.Tensor]:
         H, tag = self.heads, L._DTYPE[span.dtype]
         a = span.empty(self.n_in)
         L.linear(h, self.w_in, self.width, self.n_in, a)
@@ -157,13 +195,13 @@ class LatentAttention:
                            pos0=span.pos0, **self._sizes(cache, cos_sin))
         y = torch.empty(span.rows, self.n_out, dtype=torch.float32, device=span.device)
         L.linear(att, self.w_out, H * self.vdim, self.n_out, y)
-        return y
+        return [y]
 
     def buffers(self) -> dict[str, int]:
         """fp32 scratch of the decode step, in elements."""
         return {"a": self.n_in, "q": self.n_q, "o": self.heads * self.vdim, "y": self.n_out}
 
-    def decode(self, chain, s: "LayeredSession", cache: LatentCache, cos_sin) -> torch.Tensor:
+    def decode(self, chain, s: "LayeredSession", cache: LatentCache, cos_sin) -> list[torch.Tensor]:
         a, q, o, y = s.buf["a"], s.buf["q"], s.buf["o"], s.buf["y"]
         chain(self.w_in, self.n_in, self.width, a)
         L.matvec(self.w_uq, self.n_q, self.q_rank, a, q, norm=L.NORM_RMS, eps=self.eps, norm_w=self.q_norm, x_offset=self.q_off)
@@ -172,7 +210,7 @@ class LatentAttention:
                         cache_dtype=L._DTYPE[cache.rows.dtype], B=1, ldq=q.numel(), lda=a.numel(), kv_off=self.kv_off, g_off=self.g_off,
                         ldu=self.w_ukv.stride(0), ldo=o.numel(), **self._sizes(cache, cos_sin))
         L.matvec(self.w_out, self.n_out, self.heads * self.vdim, o, y)
-        return y
+        return [y]
 
 
 class GatedLinearAttention:
@@ -198,11 +236,11 @@ class GatedLinearAttention:
 
     def _args(self, p: torch.Tensor, ldp: int, out: torch.Tensor, ldo: int, state: RecurrentState, dtype: torch.dtype, B: int, T: int) -> dict:
         return dict(p=p.data_ptr(), out=out.data_ptr(), state=state.s.data_ptr(), a2=self.w_a2.data_ptr(), a2_b=self.a2_bias.data_ptr(),
-                    norm_w=self.norm_w.data_ptr(), tau=self.tau, eps=self.eps, dtype=L._DTYPE[dtype], B=B, T=T, H=self.heads, dim=self.dim,
+                    norm_w=self.norm_w.data_ptr(), tau=self.tau, eps=self.eps, kind=L.GLA_LOW_RANK, dtype=L._DTYPE[dtype], B=B, T=T, H=self.heads, dim=self.dim,
                     vdim=self.vdim, ldp=ldp, q_off=self.q_off, k_off=self.k_off, v_off=self.v_off, g_off=self.g_off, a_off=self.a_off,
                     a_rank=self.a_rank, lda2=self.w_a2.stride(0), lds=state.s.shape[3], ldo=ldo)
 
-    def prompt(self, h: torch.Tensor, span: Span, state: RecurrentState, cos_sin) -> torch.Tensor:
+    def prompt(self, h: torch.Tensor, span: Span, state: RecurrentState, cos_sin) -> list[torch.Tensor]:
         p = span.empty(self.n_in)
         L.linear(h, self.w_in, self.width, self.n_in, p)
         o = span.empty(self.heads * self.vdim)
@@ -210,70 +248,313 @@ class GatedLinearAttention:
         L.gla_prefill(ws, **self._args(p, p.stride(0), o, o.stride(0), state, span.dtype, span.B, span.T))
         y = torch.empty(span.rows, self.n_out, dtype=torch.float32, device=span.device)
         L.linear(o, self.w_out, self.heads * self.vdim, self.n_out, y)
-        return y
+        return [y]
 
     def buffers(self) -> dict[str, int]:
         return {"a": self.n_in, "o": self.heads * self.vdim, "y": self.n_out}
 
-    def decode(self, chain, s: "LayeredSession", state: RecurrentState, cos_sin) -> torch.Tensor:
+    def decode(self, chain, s: "LayeredSession", state: RecurrentState, cos_sin) -> list[torch.Tensor]:
         p, o, y = s.buf["a"], s.buf["o"], s.buf["y"]
         chain(self.w_in, self.n_in, self.width, p)
         L.gla_decode(**self._args(p, p.numel(), o, o.numel(), state, torch.float32, 1, 1))
         L.matvec(self.w_out, self.n_out, self.heads * self.vdim, o, y)
-        return y
+        return [y]
+
+
+# ---------------------------------------------------------------------- branches
+class MixedHeadAttention:
+    """A branch (see `BranchMixer`): grouped attention over a sliding window without a rotation.  Scores pass through a soft
+    cap, lose r1_h ln(1 + r2_h distance) and are mixed across the heads by `talk` (heads, heads) before the softmax; the
+    heads' outputs are gated element by element by a sigmoid."""
+
+    def __init__(self, *, heads: int, kv_heads: int, dim: int, vdim: int, window: int, scale: float, softcap: float, context_len: int,
+                 w_q, w_k, w_v, w_gate, r1, r2, talk, w_out):
+        if heads % kv_heads:
+            raise ValueError(f"{heads} heads do not share {kv_heads} key/value heads evenly")
+        self.heads, self.kv_heads, self.dim, self.vdim, self.window, self.scale, self.softcap = heads, kv_heads, dim, vdim, window, scale, softcap
+        width = w_q.shape[1]
+        _shapes({"q": (w_q, (heads * dim, width)), "k": (w_k, (kv_heads * dim, width)), "v": (w_v, (kv_heads * vdim, width)),
+                 "g": (w_gate, (heads * vdim, width)), "r1": (r1, (heads,)), "r2": (r2, (heads,)), "talk": (talk, (heads, heads)),
+                 "o": (w_out, (w_out.shape[0], heads * vdim))})
+        # keys and values stand side by side, each from a multiple of eight rows on: the cache's row is a copy of them
+        self.w_in = [w_q, w_k, w_v, w_gate]
+        self.kv_cols = L.pad8(kv_heads * dim) + kv_heads * vdim
+        self.w_out, self.cols = w_out, heads * vdim
+        self.talk = talk.float().contiguous()
+        n = min(window, context_len) if window > 0 else context_len
+        far = torch.arange(n, dtype=torch.float64, device=r1.device)
+        self.penalty = (r1.double()[:, None] * torch.log1p(r2.double()[:, None] * far)).float().contiguous()
+
+    def place(self, offsets: list[int]) -> None:
+        """Columns of the pieces of w_in in the joint projection."""
+        self.q_off, self.k_off, _, self.g_off = offsets
+
+    def new_cache(self, batch: int, context_len: int, dtype, device) -> KeyValueCache:
+        return KeyValueCache(batch, context_len, self.kv_heads * self.dim, self.kv_heads * self.vdim, dtype, device)
+
+    def _sizes(self, cache: KeyValueCache) -> dict:
+        return dict(cache=cache.rows.data_ptr(), penalty=self.penalty.data_ptr(), talk=self.talk.data_ptr(), scale=self.scale, softcap=self.softcap,
+                    H=self.heads, G=self.kv_heads, dim=self.dim, vdim=self.vdim, ctx=cache.rows.shape[1], ldc=cache.rows.shape[2],
+                    v_off=cache.v_off, window=self.window, n_pen=self.penalty.shape[1])
+
+    def prompt(self, a: torch.Tensor, span: Span, cache: KeyValueCache) -> torch.Tensor:
+        """a: the joint projection of the portion's rows."""
+        o = span.empty(self.cols)
+        L.cache_append(a, self.k_off, self.kv_cols, cache.rows, span.B, span.T, span.pos0)
+        L.talk_attention(span.device, q=L._ptr(a, self.q_off), gate=L._ptr(a, self.g_off), out=o.data_ptr(), dtype=L._DTYPE[span.dtype], B=span.B,
+                         T=span.T, ldq=a.stride(0), ldg=a.stride(0), ldo=o.stride(0), pos0=span.pos0, **self._sizes(cache))
+        return o
+
+    def decode(self, a: torch.Tensor, o: torch.Tensor, s: "LayeredSession", cache: KeyValueCache) -> None:
+        L.talk_decode(p=a.data_ptr(), pos=s.pos.data_ptr(), out=o.data_ptr(), cache_dtype=L._DTYPE[cache.rows.dtype], B=1, ldp=a.numel(),
+                      q_off=self.q_off, k_off=self.k_off, g_off=self.g_off, ldo=o.numel(), **self._sizes(cache))
+
+
+class ForgetLinearAttention:
+    """A branch: the HGRN2 recurrence.  Per head a (dim x vdim) fp32 state that decays by f per channel and takes up
+    (1 - f) v^T, f = lower + (1 - lower) sigmoid(z); read by silu(q), RMS-normed per head."""
+
+    def __init__(self, *, heads: int, dim: int, vdim: int, eps: float, w_q, w_f, f_bias, lower, w_v, norm_w, w_out):
+        self.heads, self.dim, self.vdim, self.eps = heads, dim, vdim, eps
+        width = w_q.shape[1]
+        _shapes({"q": (w_q, (heads * dim, width)), "f": (w_f, (heads * dim, width)), "f.b": (f_bias, (heads * dim,)),
+                 "lower": (lower, (heads * dim,)), "v": (w_v, (heads * vdim, width)), "norm": (norm_w, (vdim,)),
+                 "o": (w_out, (w_out.shape[0], heads * vdim))})
+        self.w_in = [w_q, w_f, w_v]
+        self.w_out, self.cols = w_out, heads * vdim
+        self.f_bias, self.lower, self.norm_w = f_bias.float(), lower.float(), norm_w.float()
+
+    def place(self, offsets: list[int]) -> None:
+        self.q_off, self.f_off, self.v_off = offsets
+
+    def new_cache(self, batch: int, context_len: int, dtype, device) -> RecurrentState:
+        return RecurrentState(batch, self.heads, self.dim, self.vdim, device)
+
+    def _args(self, p: torch.Tensor, ldp: int, out: torch.Tensor, ldo: int, state: RecurrentState, dtype: torch.dtype, B: int, T: int) -> dict:
+        return dict(p=p.data_ptr(), out=out.data_ptr(), state=state.s.data_ptr(), a2_b=self.f_bias.data_ptr(), lower=self.lower.data_ptr(),
+                    norm_w=self.norm_w.data_ptr(), eps=self.eps, kind=L.GLA_FORGET, dtype=L._DTYPE[dtype], B=B, T=T, H=self.heads, dim=self.dim,
+                    vdim=self.vdim, ldp=ldp, q_off=self.q_off, k_off=self.f_off, v_off=self.v_off, g_off=-1, lds=state.s.shape[3], ldo=ldo)
+
+    def prompt(self, a: torch.Tensor, span: Span, state: RecurrentState) -> torch.Tensor:
+        o = span.empty(self.cols)
+        ws = torch.empty(L.gla_workspace_bytes(span.B, span.T, self.heads, self.dim, self.vdim), dtype=torch.uint8, device=span.device)
+        L.gla_prefill(ws, **self._args(a, a.stride(0), o, o.stride(0), state, span.dtype, span.B, span.T))
+        return o
+
+    def decode(self, a: torch.Tensor, o: torch.Tensor, s: "LayeredSession", state: RecurrentState) -> None:
+        L.gla_decode(**self._args(a, a.numel(), o, o.numel(), state, torch.float32, 1, 1))
+
+
+class BranchMixer:
+    """One or two branches side by side: one product for all their projections, every branch on its columns, an output
+    projection each.  The results stay apart; the layer's link weights and adds them."""
+
+    def __init__(self, kind: str, branches: list):
+        if not 1 <= len(branches) <= 2:
+            raise ValueError(f"{len(branches)} branches")
+        self.kind, self.branches = kind, branches
+        self.w_in, offs = L.stack_rows([m for b in branches for m in b.w_in])
+        self.width, self.n_in = branches[0].w_in[0].shape[1], self.w_in.shape[0]
+        for b in branches:
+            b.place(offs[:len(b.w_in)])
+            offs = offs[len(b.w_in):]
+            del b.w_in
+            b.w_out, b.n_out = L.pad_matrix(b.w_out), b.w_out.shape[0]
+
+    def new_cache(self, batch: int, context_len: int, dtype, device) -> BranchCaches:
+        return BranchCaches([b.new_cache(batch, context_len, dtype, device) for b in self.branches])
+
+    def prompt(self, h: torch.Tensor, span: Span, cache: BranchCaches, cos_sin) -> list[torch.Tensor]:
+        a = span.empty(self.n_in)
+        L.linear(h, self.w_in, self.width, self.n_in, a)
+        ys = []
+        for b, c in zip(self.branches, cache.parts):
+            o = b.prompt(a, span, c)
+            y = torch.empty(span.rows, b.n_out, dtype=torch.float32, device=span.device)
+            L.linear(o, b.w_out, b.cols, b.n_out, y)
+            ys.append(y)
+        return ys
+
+    def buffers(self) -> dict[str, int]:
+        out = {"a": self.n_in}
+        for i, b in enumerate(self.branches):
+            out[f"o{i}"], out[f"y{i}"] = b.cols, b.n_out
+        return out
+
+    def decode(self, chain, s: "LayeredSession", cache: BranchCaches, cos_sin) -> list[torch.Tensor]:
+        a = s.buf["a"]
+        chain(self.w_in, self.n_in, self.width, a)
+        jobs = []
+        for i, (b, c) in enumerate(zip(self.branches, cache.parts)):
+            b.decode(a, s.buf[f"o{i}"], s, c)
+            jobs.append((b.w_out, b.n_out, b.cols, s.buf[f"o{i}"], s.buf[f"y{i}"]))
+        L.matvec_pair(*jobs) if len(jobs) == 2 else L.matvec(*jobs[0])
+        return [j[4] for j in jobs]
+
+
+def _shapes(want: dict) -> None:
+    for name, (w, shape) in want.items():
+        if tuple(w.shape) != shape:
+            raise ValueError(f"{name} has shape {tuple(w.shape)}, the layer's sizes want {shape}")
 
 
 class DenseFFN:
-    """W_down (silu(W_gate h + b) * (W_up h + b)) + b; gate and up rows interleaved, so the product's epilogue emits the
-    activation."""
+    """W_down act(W_gate h + b, W_up h + b) + b with a gated activation (silu(g) * u unless told otherwise; biases may be
+    absent); gate and up rows interleaved, so the product's epilogue emits the activation."""
 
-    def __init__(self, *, w_gate, b_gate, w_up, b_up, w_down, b_down):
+    def __init__(self, *, w_gate, w_up, w_down, b_gate=None, b_up=None, b_down=None, act: L.Act = L.SWIGLU):
         F, self.width = w_gate.shape
-        self.hidden, self.n_out = F, w_down.shape[0]
+        self.hidden, self.n_out, self.act = F, w_down.shape[0], act
         self.w_gu = L.pad_matrix(torch.stack((w_gate, w_up), dim=1).reshape(2 * F, self.width))
-        self.b_gu = torch.stack((b_gate.float(), b_up.float()), dim=1).reshape(-1).contiguous()
-        self.w_down, self.b_down = L.pad_matrix(w_down), b_down.float()
+        self.b_gu = None if b_gate is None else torch.stack((b_gate.float(), b_up.float()), dim=1).reshape(-1).contiguous()
+        self.w_down, self.b_down = L.pad_matrix(w_down), None if b_down is None else b_down.float()
 
-    def prompt(self, h: torch.Tensor, span: Span) -> torch.Tensor:
+    def prompt(self, h: torch.Tensor, span: Span) -> list[torch.Tensor]:
         act = span.empty(self.hidden)
-        L.linear(h, self.w_gu, self.width, 2 * self.hidden, act, bias=self.b_gu, act=L.ACT_SWIGLU_PAIRS)
+        L.linear(h, self.w_gu, self.width, 2 * self.hidden, act, bias=self.b_gu, act=self.act)
         y = torch.empty(span.rows, self.n_out, dtype=torch.float32, device=span.device)
         L.linear(act, self.w_down, self.hidden, self.n_out, y, bias=self.b_down)
-        return y
+        return [y]
 
     def buffers(self) -> dict[str, int]:
         return {"f": self.hidden, "y": self.n_out}
 
-    def decode(self, chain, s: "LayeredSession") -> torch.Tensor:
+    def decode(self, chain, s: "LayeredSession") -> list[torch.Tensor]:
         f, y = s.buf["f"], s.buf["y"]
-        chain(self.w_gu, 2 * self.hidden, self.width, f, bias=self.b_gu, act=L.ACT_SWIGLU_PAIRS)
+        chain(self.w_gu, 2 * self.hidden, self.width, f, bias=self.b_gu, act=self.act)
         L.matvec(self.w_down, self.n_out, self.hidden, f, y, bias=self.b_down)
-        return y
+        return [y]
 
 
+# ---------------------------------------------------------------------- the residual
 @dataclass
-class Layer:
-    mixer: LatentAttention | GatedLinearAttention
-    norm1: torch.Tensor                     # before and after the mixer
-    norm1_post: torch.Tensor
-    ffn: DenseFFN | None = None
-    norm2: torch.Tensor | None = None       # before and after the feed-forward
-    norm2_post: torch.Tensor | None = None
+class Link:
+    """How a sublayer hangs on the residual.  One stream: x <- x + norm(y) * post around h = norm(x) * norm.  Hyper-connections:
+    h = norm(sum_s read_s x_s) * norm, y = the sum of the results (each normed by `post_norm`, if given) times their weights
+    in `post`, then x_t <- sum_s mix[s, t] x_s + share_t y, all streams at once."""
+    norm: torch.Tensor                      # (C) weight of the norm in front
+    post: list[torch.Tensor] = field(default_factory=list)       # (C) weight of each result
+    post_norm: str | None = None
+    read: torch.Tensor | None = None
+    share: torch.Tensor | None = None
+    mix: torch.Tensor | None = None
+
+    def behind(self, before: "Link | None") -> torch.Tensor:
+        """The coefficients of the step from the link `before` to this one (nb_stream_args): what this link reads, expressed in
+        the streams in front of `before`'s update and its result."""
+        read = self.read.double()
+        n = read.numel()
+        if before is None:
+            read, direct, share, mix = read, read.new_zeros(1), read.new_zeros(n), torch.eye(n, dtype=read.dtype, device=read.device)
+        else:
+            share, mix = before.share.double(), before.mix.double()
+            read, direct = mix @ read, (share @ read).reshape(1)
+        return torch.cat([read, direct, share, mix.reshape(-1)]).float()
+
+
+class PromptResidual:
+    """The residual of a portion of a prompt: `enter` applies what the sublayer before left and returns the next one's input."""
+
+    def __init__(self, model: "LayeredDecoder", tokens: torch.Tensor, span: Span):
+        self.m, self.span = model, span
+        self.x = torch.empty(span.rows, *([model.streams] if model.streams else []), model.width, dtype=torch.float32, device=span.device)
+        L.embed_scaled(model.embedding, tokens.contiguous(), model.embedding_scale, self.x)
+        self.h = span.empty(model.width)
+        self.ys, self.link, self.n = [], None, 0
+
+    def leave(self, link: Link, ys: list[torch.Tensor]) -> None:
+        self.ys, self.link = ys, link
+
+    def keep(self, rows: list[int]) -> None:
+        """Only these rows go on."""
+        if len(rows) == 1:
+            pick = slice(rows[0], rows[0] + 1)
+            self.x, self.ys = self.x[pick], [y[pick] for y in self.ys]
+        else:
+            at = torch.tensor(rows, dtype=torch.long, device=self.x.device)
+            self.x, self.ys = self.x.index_select(0, at), [y.index_select(0, at) for y in self.ys]
+        self.h = L.rows_empty(len(rows), self.m.width, self.span.dtype, self.x.device)
+
+    def enter(self, link: Link) -> torch.Tensor:
+        y, post = (self.ys[0], self.link.post[0]) if self.ys else (None, None)
+        L.residual_norm(self.x, y, post, link.norm, NORMS[self.m.norm], self.m.eps, self.h)
+        return self.h
+
+    def total(self) -> torch.Tensor:
+        """The residual after `enter`, (rows, C)."""
+        return self.x.clone()
+
+
+class PromptStreams(PromptResidual):
+    """The same with hyper-connections: x (rows, streams, C)."""
+
+    def enter(self, link: Link) -> torch.Tensor:
+        L.stream_norm(self.x, self.ys, self.link.post if self.ys else [], self.m.post_norm(self.link), self.m.coefs[self.n], NORMS[self.m.norm],
+                      self.m.eps, link.norm, self.h)
+        self.n += 1
+        return self.h
+
+    def total(self) -> torch.Tensor:
+        return self.x.sum(1)
+
+
+class DecodeResidual:
+    """The residual of a decode step of one sequence, in a session's two buffers; `chain` makes the product that follows, with
+    the residual's update and the norm folded in."""
+
+    def __init__(self, model: "LayeredDecoder", s: "LayeredSession"):
+        self.m, self.xa, self.xb = model, s.buf["x"], s.buf["x2"]
+        L.embed_scaled(model.embedding, s.token, model.embedding_scale, self.xa.view(1, *([model.streams] if model.streams else []), model.width))
+        self.ys, self.link, self.n = [], None, 0
+
+    def leave(self, link: Link, ys: list[torch.Tensor]) -> None:
+        self.ys, self.link = ys, link
+
+    def chain(self, link: Link):
+        def run(w, n, k, out, bias=None, act=L.PLAIN):
+            opt = dict(bias=bias, act=act, norm=NORMS[self.m.norm], eps=self.m.eps, norm_w=link.norm)
+            if not self.ys:
+                L.matvec(w, n, k, self.xa, out, **opt)
+            else:
+                L.matvec(w, n, k, self.xa, out, delta=self.ys[0], delta_w=self.link.post[0], x_out=self.xb, **opt)
+                self.xa, self.xb = self.xb, self.xa
+        return run
+
+
+class DecodeStreams(DecodeResidual):
+    def chain(self, link: Link):
+        def run(w, n, k, out, bias=None, act=L.PLAIN):
+            shape = (self.m.streams, self.m.width)
+            L.matvec_streams(w, n, k, out, self.xa.view(shape), self.xb.view(shape), self.ys, self.link.post if self.ys else [],
+                             self.m.post_norm(self.link), self.m.coefs[self.n], NORMS[self.m.norm], self.m.eps, link.norm, bias, act)
+            if self.ys:
+                self.xa, self.xb = self.xb, self.xa
+            self.n += 1
+        return run
 
 
 # ---------------------------------------------------------------------- model and session
+@dataclass
+class Layer:
+    mixer: LatentAttention | GatedLinearAttention | BranchMixer
+    link1: Link                             # around the mixer
+    ffn: DenseFFN | None = None
+    link2: Link | None = None               # around the feed-forward
+
+
 @dataclass
 class LayeredDecoder:
     """Embedding (scaled) -> layers -> norm -> head.  `context_len` bounds a sequence's positions."""
     embedding: torch.Tensor                 # (V, C) bf16
     embedding_scale: float
     layers: list[Layer]
-    final_norm: torch.Tensor
+    final: Link
     head: torch.Tensor                      # (V, C) bf16, padded columns
     norm: str                               # "layer" | "rms"
     eps: float
     dtype: torch.dtype
     context_len: int
+    streams: int = 0                        # streams of hyper-connections; 0: one residual with norms behind the sublayers
     _tables: dict = field(default_factory=dict)
 
     def __post_init__(self):
@@ -286,6 +567,12 @@ class LayeredDecoder:
                 raise ValueError(f"layer {i} reads the cache of layer {src}, which is not an earlier latent-attention layer with its own")
             if (other.rank, other.rot) != (layer.mixer.rank, layer.mixer.rot):
                 raise ValueError(f"layer {i} reads the cache of layer {src}, whose latent size or rotation differs")
+        links = [k for layer in self.layers for k in (layer.link1, layer.link2) if k is not None] + [self.final]
+        self.coefs = [k.behind(links[i - 1] if i else None) for i, k in enumerate(links)] if self.streams else []
+
+    @staticmethod
+    def post_norm(link: Link | None) -> int | None:
+        return None if link is None or link.post_norm is None else NORMS[link.post_norm]
 
     @property
     def width(self) -> int:
@@ -325,41 +612,27 @@ class LayeredDecoder:
         """tokens (B, T) at positions pos0 .. -> logits (B, len(want), V) fp32 of the places `want`; caches and states are
         updated.  trace: a list that receives the residual stream (B, T, C) after every layer."""
         B, T = tokens.shape
-        norm, eps, C = NORMS[self.norm], self.eps, self.width
         span = Span(B, T, pos0, self.dtype, self.device)
-        x = torch.empty(span.rows, C, dtype=torch.float32, device=self.device)
-        L.embed_scaled(self.embedding, tokens.contiguous(), self.embedding_scale, x)
-        h = span.empty(C)
-        y, post = None, None
-        for layer, cache in zip(self.layers, caches):
-            L.residual_norm(x, y, post, layer.norm1, norm, eps, h)
-            if trace is not None and y is not None:
-                trace.append(x.view(B, T, C).clone())
-            y, post = layer.mixer.prompt(h, span, cache, self.tables(layer.mixer)), layer.norm1_post
+        res = (PromptStreams if self.streams else PromptResidual)(self, tokens, span)
+        for i, (layer, cache) in enumerate(zip(self.layers, caches)):
+            h = res.enter(layer.link1)
+            if trace is not None and i:
+                trace.append(res.total().view(B, T, -1))
+            res.leave(layer.link1, layer.mixer.prompt(h, span, cache, self.tables(layer.mixer)))
             if layer.ffn is not None:
-                L.residual_norm(x, y, post, layer.norm2, norm, eps, h)
-                y, post = layer.ffn.prompt(h, span), layer.norm2_post
-        if trace is None and len(want) < T:  # the last norm and the head run on the wanted rows only
-            if not want:
-                return torch.empty(B, 0, self.vocab_size, dtype=torch.float32, device=self.device)
-            if B == 1 and len(want) == 1:
-                x, y = x[want[0]:want[0] + 1], y[want[0]:want[0] + 1]
-            else:
-                rows = torch.tensor([b * T + w for b in range(B) for w in want], dtype=torch.long, device=self.device)
-                x, y = x.index_select(0, rows), y.index_select(0, rows)
-            return self._head(x, y, post).view(B, len(want), -1)
-        logits = self._head(x, y, post).view(B, T, -1)
-        if trace is not None:
-            trace.append(x.view(B, T, C).clone())
-        return logits[:, want, :]
-
-    def _head(self, x, y, post) -> torch.Tensor:
-        rows = x.shape[0]
-        h = L.rows_empty(rows, self.width, self.dtype, self.device)
-        L.residual_norm(x, y, post, self.final_norm, NORMS[self.norm], self.eps, h)
-        logits = torch.empty(rows, self.vocab_size, dtype=torch.float32, device=self.device)
+                res.leave(layer.link2, layer.ffn.prompt(res.enter(layer.link2), span))
+        some = trace is None and len(want) < T          # the last norm and the head run on the wanted rows only
+        if some and not want:
+            return torch.empty(B, 0, self.vocab_size, dtype=torch.float32, device=self.device)
+        if some:
+            res.keep([b * T + w for b in range(B) for w in want])
+        h = res.enter(self.final)
+        logits = torch.empty(h.shape[0], self.vocab_size, dtype=torch.float32, device=self.device)
         L.linear(h, self.head, self.width, self.vocab_size, logits)
-        return logits
+        if trace is not None:
+            trace.append(res.total().view(B, T, -1))
+        logits = logits.view(B, -1, self.vocab_size)
+        return logits if some else logits[:, want, :]
 
 
 class LayeredSession(Session):
@@ -371,7 +644,8 @@ class LayeredSession(Session):
         self.caches = model.new_caches(batch_size)
         for layer in model.layers:           # tables are built before anything is captured
             model.tables(layer.mixer)
-        sizes: dict[str, int] = {"x": model.width, "x2": model.width}
+        stream = max(1, model.streams) * model.width
+        sizes: dict[str, int] = {"x": stream, "x2": stream}
         for layer in model.layers:
             for part in (layer.mixer, layer.ffn):
                 for name, n in (part.buffers() if part is not None else {}).items():
@@ -385,7 +659,7 @@ class LayeredSession(Session):
             cache.reset()
 
     def _step_state(self) -> list[torch.Tensor]:
-        return [c.s for c in self.caches if isinstance(c, RecurrentState)]
+        return [t for c in {id(c): c for c in self.caches}.values() for t in c.carried()]
 
     def _prefill_body(self, prompt: torch.Tensor) -> None:
         self._on_reset()
@@ -411,26 +685,12 @@ class LayeredSession(Session):
             self._take(m.forward(self.token, self.pos_host, self.caches, [0]))
             self.pos.add_(1)
             return
-        norm, eps = NORMS[m.norm], m.eps
-        xa, xb = self.buf["x"], self.buf["x2"]                  # the residual stream, ping-pong
-        L.embed_scaled(m.embedding, self.token, m.embedding_scale, xa.view(1, -1))
-        y, post = None, None
-
-        def chain(norm_w):
-            """The next product of the chain: x += post-norm(y), then w . norm(x)."""
-            def run(w, n, k, out, bias=None, act=L.ACT_NONE):
-                nonlocal xa, xb
-                if y is None:
-                    L.matvec(w, n, k, xa, out, bias=bias, act=act, norm=norm, eps=eps, norm_w=norm_w)
-                else:
-                    L.matvec(w, n, k, xa, out, bias=bias, act=act, norm=norm, eps=eps, norm_w=norm_w, delta=y, delta_w=post, x_out=xb)
-                    xa, xb = xb, xa
-            return run
+        res = (DecodeStreams if m.streams else DecodeResidual)(m, self)
         for layer, cache in zip(m.layers, self.caches):
-            y, post = layer.mixer.decode(chain(layer.norm1), self, cache, m.tables(layer.mixer)), layer.norm1_post
+            res.leave(layer.link1, layer.mixer.decode(res.chain(layer.link1), self, cache, m.tables(layer.mixer)))
             if layer.ffn is not None:
-                y, post = layer.ffn.decode(chain(layer.norm2), self), layer.norm2_post
-        chain(m.final_norm)(m.head, m.vocab_size, m.width, self.logits)
+                res.leave(layer.link2, layer.ffn.decode(res.chain(layer.link2), self))
+        res.chain(m.final)(m.head, m.vocab_size, m.width, self.logits)
         L.argmax(self.logits, self.token, self.pos)
 
     def check(self) -> None:

@@ -5,9 +5,9 @@ from __future__ import annotations
 
 import torch
 
-from .layered import DenseFFN, GatedLinearAttention, LatentAttention, Layer, LayeredDecoder, Rotation, Yarn
+from .layered import DenseFFN, GatedLinearAttention, LatentAttention, Layer, LayeredDecoder, Link, Rotation, Yarn
 from .layer_ops import pad_matrix
-from .weights import Checkpoint
+from .weights import load_checkpoint
 
 
 def _rotation(rot: dict) -> Rotation:
@@ -60,19 +60,14 @@ def build(config: dict, tensor, dtype: torch.dtype, context_len: int) -> Layered
         norm = lambda name: tensor(f"l{i}.{name}", (C,)).float()                                        # noqa: E731
         mixer = MIXERS[spec["type"]](lambda n, s: tensor(f"l{i}.mix.{n}", s), spec["mixer"], C, eps)
         ffn = _ffn(lambda n, s: tensor(f"l{i}.mlp.{n}", s), spec["mlp"], C)
-        extra = {} if ffn is None else {"ffn": ffn, "norm2": norm("norm2"), "norm2_post": norm("norm2b")}
-        layers.append(Layer(mixer, norm("norm1"), norm("norm1b"), **extra))
-    return LayeredDecoder(tensor("embed", (V, C)), float(config["embedding"]["scale"]), layers, tensor("final.norm", (C,)).float(),
+        extra = {} if ffn is None else {"ffn": ffn, "link2": Link(norm("norm2"), [norm("norm2b")])}
+        layers.append(Layer(mixer, Link(norm("norm1"), [norm("norm1b")]), **extra))
+    return LayeredDecoder(tensor("embed", (V, C)), float(config["embedding"]["scale"]), layers, Link(tensor("final.norm", (C,)).float()),
                           pad_matrix(tensor("head", (V, C))), "layer", eps, dtype, context_len)
 
 
 def load(folder: str, config: dict, dtype: torch.dtype, context_len: int, device) -> LayeredDecoder:
-    ckpt = Checkpoint(f"{folder}/model.safetensors", device)
-    model = build(config, lambda n, s: ckpt.get(n, s), dtype, context_len)
-    if ckpt.unread():
-        raise ValueError(f"the checkpoint has tensors that the configuration does not name: {ckpt.unread()[:8]}")
-    torch.cuda.synchronize(device)           # the kernels request weights before they wait for earlier work of the stream
-    return model
+    return load_checkpoint(folder, device, lambda tensor: build(config, tensor, dtype, context_len))
 
 
 def random_tensors(config: dict, seed: int, device) -> dict[str, torch.Tensor]:

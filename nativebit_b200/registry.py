@@ -29,6 +29,7 @@ FAMILIES: dict[str, Family] = {
     # fp32 activations enter the packed products as two fp16 terms: not a 32-bit mode
     "PackedGPT": Family("packed", "nativebit_b200.generate", "load_folder", ("bfloat16",)),
     "Nerulorn": Family("layered", "nativebit_b200.nerulorn", "load"),
+    "Nabalix": Family("layered", "nativebit_b200.nabalix", "load"),
 }
 
 

@@ -51,6 +51,16 @@ class Checkpoint:
         return sorted(set(self._index) - self._read)
 
 
+def load_checkpoint(folder: str, device, build):
+    """build(tensor) with tensor(name, shape) -> the weight on the device; every tensor of the file must be asked for."""
+    ckpt = Checkpoint(f"{folder}/model.safetensors", device)
+    model = build(lambda n, s: ckpt.get(n, s))
+    if ckpt.unread():
+        raise ValueError(f"the checkpoint has tensors that the configuration does not name: {ckpt.unread()[:8]}")
+    torch.cuda.synchronize(device)           # the kernels request weights before they wait for earlier work of the stream
+    return model
+
+
 def write_safetensors(path: str, tensors: dict[str, torch.Tensor]) -> None:
     """The writer's side of the format (exporters, tests)."""
     names = {v[1]: k for k, v in _TYPES.items()}

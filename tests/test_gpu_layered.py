@@ -111,7 +111,7 @@ def test_linear(dev, m, n, k, dtype):
         y = x @ w.T + b
         ref = O.silu(y[:, ::2]) * y[:, 1::2]
         act = L.rows_empty(m, n // 2, dtype, dev)
-        L.linear(xt, wt, k, n, act, bias=cu(b), act=L.ACT_SWIGLU_PAIRS)
+        L.linear(xt, wt, k, n, act, bias=cu(b), act=L.SWIGLU)
         close(act[:, :n // 2], ref, max(TOL[dtype], 1e-5))
 
 
@@ -139,7 +139,7 @@ def test_matvec(dev, n, k):
     if n % 2 == 0:
         z = w @ x.astype(np.float64) + b
         act = torch.empty(n // 2, device=dev)
-        L.matvec(wt, n, k, cu(x), act, bias=cu(b), act=L.ACT_SWIGLU_PAIRS)
+        L.matvec(wt, n, k, cu(x), act, bias=cu(b), act=L.SWIGLU)
         close(act, O.silu(z[::2]) * z[1::2], 1e-5)
 
 

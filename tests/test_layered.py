@@ -191,17 +191,17 @@ def test_layered_argument_checks_need_no_gpu(layered_lib):
     from nativebit_b200 import _lib
     l = _lib.layered_lib()
     fake, odd = 4096, 4100
-    assert l.nb_embed_scaled(None, fake, 1, 8, 8, 1.0, fake, None) == 1
+    assert l.nb_embed_scaled(None, fake, 1, 8, 8, 1.0, 1, fake, None) == 1
     assert l.nb_residual_norm(fake, fake, None, fake, 1, 1e-6, fake, 0, 8, 1, 8, None) == 1          # y without its weight
     assert l.nb_residual_norm(fake, None, None, fake, 2, 1e-6, fake, 0, 8, 1, 8, None) == 1          # unknown norm
     assert l.nb_residual_norm(fake, None, None, fake, 1, 1e-6, fake, 0, 20000, 1, 20000, None) == 3  # row too long
-    assert l.nb_linear_bf16(fake, 12, fake, 16, None, 0, 4, 8, 12, fake, 2, 8, None, None) == 2      # row stride no multiple of 8
-    assert l.nb_linear_bf16(fake, 16, fake, 16, None, 1, 4, 7, 12, fake, 2, 8, None, None) == 3      # pairs need an even N
-    assert l.nb_linear_bf16(odd, 16, fake, 16, None, 0, 4, 8, 12, fake, 2, 8, None, None) == 2
-    assert l.nb_linear_f32(fake, 8, fake, 8, None, 0, 4, 8, 12, fake, 8, None) == 1                  # stride below K
-    a = _lib.MatvecArgs(fake, None, fake, fake, fake, fake, fake, fake, 1e-6, 8, 8, 8, 0, 1)
+    assert l.nb_linear_bf16(fake, 12, fake, 16, None, 0, 0.0, 0.0, 4, 8, 12, fake, 2, 8, None, None) == 2      # row stride no multiple of 8
+    assert l.nb_linear_bf16(fake, 16, fake, 16, None, 1, 0.0, 0.0, 4, 7, 12, fake, 2, 8, None, None) == 3      # pairs need an even N
+    assert l.nb_linear_bf16(odd, 16, fake, 16, None, 0, 0.0, 0.0, 4, 8, 12, fake, 2, 8, None, None) == 2
+    assert l.nb_linear_f32(fake, 8, fake, 8, None, 0, 0.0, 0.0, 4, 8, 12, fake, 8, None) == 1                  # stride below K
+    a = _lib.MatvecArgs(fake, None, fake, fake, fake, fake, fake, fake, 1e-6, 0.0, 0.0, 8, 8, 8, 0, 1)
     assert l.nb_matvec_bf16(ctypes.byref(a), None) == 1                                              # x_out aliases x
-    a = _lib.MatvecArgs(fake, None, fake, fake, None, None, None, None, 0.0, 8, 9, 12, 0, 0)
+    a = _lib.MatvecArgs(fake, None, fake, fake, None, None, None, None, 0.0, 0.0, 0.0, 8, 9, 12, 0, 0)
     assert l.nb_matvec_bf16(ctypes.byref(a), None) == 2
     g = dict(p=fake, out=fake, state=fake, a2=fake, a2_b=fake, norm_w=fake, tau=4.0, eps=1e-6, dtype=0, B=1, T=1, H=2, dim=8, vdim=6, ldp=64,
              q_off=0, k_off=16, v_off=32, g_off=44, a_off=56, a_rank=4, lda2=8, lds=8, ldo=16)
