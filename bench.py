@@ -917,13 +917,20 @@ def main():
     ap.add_argument("--layered", action="store_true",
                     help="instead of the default workload: prefill and decode throughput of the layered decoder beside the packed "
                          "one, and every kernel of both against its roofline")
-    ap.add_argument("--layered-sizes", default="1024,2048,2560", help="widths of --layered")
-    ap.add_argument("--layered-prompts", type=int, nargs="+", default=[512, 2048, 4096], help="prompt lengths of --layered")
-    ap.add_argument("--no-layered-kernels", action="store_true", help="--layered without the per-kernel table")
+    ap.add_argument("--nabalix", action="store_true",
+                    help="instead of the default workload: prefill and decode throughput of Nabalix layers beside Nerulorn's, and every "
+                         "kernel of both against its roofline")
+    ap.add_argument("--nabalix-only", default="", metavar="KERNEL", help="--nabalix: time this kernel only")
+    ap.add_argument("--layered-sizes", default="1024,2048,2560", help="widths of --layered and --nabalix")
+    ap.add_argument("--layered-prompts", type=int, nargs="+", default=[512, 2048, 4096], help="prompt lengths of --layered and --nabalix")
+    ap.add_argument("--no-layered-kernels", action="store_true", help="--layered or --nabalix without the per-kernel table")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3)
     if args.layered:
         from nativebit_b200.bench_layered import run
+        return run(args)
+    if args.nabalix or args.nabalix_only:
+        from nativebit_b200.bench_nabalix import run
         return run(args)
     if args.decode_only:
         run_decode_only(args)
