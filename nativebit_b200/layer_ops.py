@@ -184,13 +184,18 @@ def cache_append(src: torch.Tensor, offset: int, cols: int, cache: torch.Tensor,
 TALK_WORKSPACE = 96 << 20              # bytes of mixed scores at a time (a block of query tiles): they stay in L2
 
 
+def talk_workspace_bytes(b: int, t: int, heads: int, pos0: int, window: int, tiles: int) -> int:
+    return int(_lib.layered_lib().nb_talk_attention_workspace_bytes(b, t, heads, pos0, window, tiles))
+
+
+def talk_attention_in(workspace: torch.Tensor, args: "_lib.TalkAttentionArgs") -> None:
+    _call("nb_talk_attention", ctypes.byref(args), workspace.data_ptr(), workspace.numel(), _stream())
+
+
 def talk_attention(device, **kw) -> None:
-    l = _lib.layered_lib()
     size = [kw[n] for n in ("B", "T", "H", "pos0", "window")]
-    one = int(l.nb_talk_attention_workspace_bytes(*size, 1))
-    n = int(l.nb_talk_attention_workspace_bytes(*size, max(1, TALK_WORKSPACE // max(one, 1))))
-    ws = torch.empty(max(n, 1), dtype=torch.uint8, device=device)
-    _call("nb_talk_attention", ctypes.byref(_lib.TalkAttentionArgs(**kw)), ws.data_ptr(), n, _stream())
+    tiles = max(1, TALK_WORKSPACE // max(1, talk_workspace_bytes(*size, 1)))
+    talk_attention_in(torch.empty(talk_workspace_bytes(*size, tiles), dtype=torch.uint8, device=device), _lib.TalkAttentionArgs(**kw))
 
 
 def talk_decode(**kw) -> None:
