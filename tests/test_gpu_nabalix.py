@@ -183,8 +183,8 @@ def test_talk_attention(dev, shape, dtype, T, pos0, window, tiles):
     for dst, lo, hi in ((cache, first, pos0), (src.view(B, T, -1), pos0, N)):               # earlier rows sit in the cache
         at = 0 if dst is cache else off
         rows = dst[:, first:pos0] if dst is cache else dst
-        rows[:, :, at:at + G * D] = cu(k[:, lo:hi].reshape(B, hi - lo, -1), dtype)
-        rows[:, :, at + v_off:at + cols] = cu(v[:, lo:hi].reshape(B, hi - lo, -1), dtype)
+        rows[:, :, at:at + G * D] = cu(k[:, lo:hi].reshape(B, hi - lo, G * D), dtype)
+        rows[:, :, at + v_off:at + cols] = cu(v[:, lo:hi].reshape(B, hi - lo, G * V), dtype)
     L.cache_append(src, off, cols, cache, B, T, pos0)
     assert torch.equal(cache[:, pos0:N, :G * D], src.view(B, T, -1)[:, :, off:off + G * D])
     assert torch.equal(cache[:, pos0:N, v_off:cols], src.view(B, T, -1)[:, :, off + v_off:off + cols])
