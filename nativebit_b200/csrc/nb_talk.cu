@@ -46,39 +46,38 @@ __device__ __forceinline__ float soft_cap_fast(float x, float cap2, float cap) {
   return cap - __fdividef(2.f * cap, 1.f + ex2(x * cap2));
 }
 
-// bf16.  A CTA of eight warps owns 64 queries x 16 NB keys of all heads: the raw scores of every head of a pair stay in the
-// registers of one thread (warp: 16 queries x 8 NB keys), where the heads are mixed.  HM >= H.
-constexpr int kScThreads = 256;
+// bf16.  A CTA of eight warps owns 16 queries, whose rows of all heads stay in shared memory, and walks `chunk` steps of
+// 64 NB keys; a step's keys arrive one key/value head at a time through a ring of `stages`.  A warp takes 8 NB of the keys:
+// the raw scores of every head of a pair stay in the registers of one thread, where the heads are mixed.  HM >= H;
+// kTwo: two heads of a group at a time share the key fragments (an even number of heads per group).
+constexpr int kScThreads = 256, kSq = 16;
 
-template <int HM, int NB>
-__global__ void __launch_bounds__(kScThreads, 1) talk_scores_bf16_kernel(const nb_talk_attention_args p, TalkBlock blk, int dk16, int vec) {
+template <int HM, int NB, bool kTwo>
+__global__ void __launch_bounds__(kScThreads, 1) talk_scores_bf16_kernel(const nb_talk_attention_args p, TalkBlock blk, int dk16, int chunk, int stages,
+                                                                         int vec) {
   extern __shared__ __align__(16) bf16 tsm[];
-  constexpr int KW = 16 * NB, kPen = kQT + KW;
-  const int dkp = dk16 + 8;
-  bf16* q_s = tsm;                       // [2][64][dkp]
-  bf16* k_s = q_s + 2 * kQT * dkp;       // [2][KW][dkp]
-  float* talk_s = reinterpret_cast<float*>(k_s + 2 * KW * dkp);   // [H][HM]
-  float* pen_s = talk_s + p.H * HM;      // [H][kPen], by distance from dmin
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, wq = warp & 3, wk = warp >> 2;
-  const int tile = blk.tile0 + blockIdx.y, q0 = tile * kQT, b = blockIdx.z;
+  constexpr int KW = 64 * NB, kPen = kSq + KW, R = kTwo ? 2 : 1;
+  const int dkp = dk16 + 8, H = p.H, D = p.dim, rep = H / p.G;
+  bf16* q_s = tsm;                       // [H][16][dkp]
+  bf16* k_s = q_s + H * kSq * dkp;       // [stages][KW][dkp]
+  float* talk_s = reinterpret_cast<float*>(k_s + stages * KW * dkp);   // [H][HM]
+  float* pen_s = talk_s + H * HM;        // [H][kPen]: of a step, by distance from its smallest
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int sub = gridDim.y - 1 - blockIdx.y, local = sub / (kQT / kSq), r0 = (sub & (kQT / kSq - 1)) * kSq, b = blockIdx.z;   // longest first
+  const int q0 = (blk.tile0 + local) * kQT;
   const int first = talk_first_key(p.pos0, q0, p.window), last = p.pos0 + min(q0 + kQT - 1, p.T - 1);
-  const int k0 = first + blockIdx.x * KW;
-  if (k0 >= first + ((last - first) / kKT + 1) * kKT) return;      // past the tile's last block of keys
-  const int rep = p.H / p.G, D = p.dim;
+  const int span = ((last - first) / kKT + 1) * kKT;               // what the tile's readers take
+  const int c0 = blockIdx.x * chunk * KW, steps = min(chunk, (span - c0 + KW - 1) / KW);
+  if (steps <= 0 || q0 + r0 >= p.T) return;
   const bf16* q = reinterpret_cast<const bf16*>(p.q);
   const bf16* cache = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.ctx * p.ldc;
-  for (int i = tid; i < 2 * (kQT + KW) * (dkp - D); i += kScThreads) {     // columns past dim stay zero
+  for (int i = tid; i < (H * kSq + stages * KW) * (dkp - D); i += kScThreads) {      // columns past dim stay zero
     const int r = i / (dkp - D);
     q_s[r * dkp + D + i - r * (dkp - D)] = from_f<bf16>(0.f);
   }
-  for (int i = tid; i < p.H * HM; i += kScThreads) {
+  for (int i = tid; i < H * HM; i += kScThreads) {
     const int h = i / HM, g = i - h * HM;
-    talk_s[i] = g < p.H ? p.talk[h * p.H + g] : 0.f;
-  }
-  const int dmin = p.pos0 + q0 - (k0 + KW - 1);
-  for (int i = tid; i < p.H * kPen; i += kScThreads) {
-    const int h = i / kPen, d = dmin + i - h * kPen;
-    pen_s[i] = p.penalty && d >= 0 && d < p.n_pen ? p.penalty[(size_t)h * p.n_pen + d] : 0.f;
+    talk_s[i] = g < H ? p.talk[h * H + g] : 0.f;
   }
   auto copy = [&](bf16* dst, int rows, auto row_of) {
     if (vec) {
@@ -98,90 +97,118 @@ __global__ void __launch_bounds__(kScThreads, 1) talk_scores_bf16_kernel(const n
       }
     }
   };
-  auto fetch = [&](int h) {              // head h's queries, and the keys if its group begins
-    copy(q_s + (h & 1) * kQT * dkp, kQT, [&](int r) { return q + (size_t)(b * p.T + min(q0 + r, p.T - 1)) * p.ldq + h * D; });
-    if (h % rep == 0) {
-      const int g = h / rep;
-      copy(k_s + (g & 1) * KW * dkp, KW, [&](int r) { return k0 + r <= last ? cache + (size_t)(k0 + r) * p.ldc + g * D : nullptr; });
+  const int items = steps * p.G;         // (step, key/value head) in order; item i uses stage i % stages
+  int ni = 0, ng = 0, ns = 0, nk = first + c0;                     // next item to request: its number, head, stage, first key
+  auto fetch = [&]() {
+    if (ni < items) {
+      const int g = ng, k0 = nk;
+      copy(k_s + ns * KW * dkp, KW, [&](int r) { return k0 + r <= last ? cache + (size_t)(k0 + r) * p.ldc + g * D : nullptr; });
+      ++ni;
+      if (++ng == p.G) { ng = 0; nk += KW; }
+      if (++ns == stages) ns = 0;
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  fetch(0);
-  const int rowa = wq * 16 + (lane >> 2), kc = wk * 8 * NB + (lane & 3) * 2;   // this lane's first query row and key column
+  auto penalties = [&](int k0) {
+    const int dmin = p.pos0 + q0 + r0 - (k0 + KW - 1);
+    for (int i = tid; i < H * kPen; i += kScThreads) {
+      const int h = i / kPen, d = dmin + i - h * kPen;
+      pen_s[i] = p.penalty && d >= 0 && d < p.n_pen ? p.penalty[(size_t)h * p.n_pen + d] : 0.f;
+    }
+  };
+  copy(q_s, H * kSq, [&](int r) { return q + (size_t)(b * p.T + min(q0 + r0 + (r & (kSq - 1)), p.T - 1)) * p.ldq + (r / kSq) * D; });
+  for (int i = 0; i + 1 < stages; ++i) fetch();                    // the queries travel with the first
+  penalties(first + c0);
+  const int rowa = lane >> 2, kc = warp * 8 * NB + (lane & 3) * 2; // this lane's first query row and key column
   const float sx = p.softcap > 0.f ? p.scale / p.softcap : p.scale, cap2 = 2.f * 1.4426950408889634f;
-  float s[HM][NB][4];
+  const int pa = p.pos0 + q0 + r0 + rowa, plast = p.pos0 + p.T - 1;
+  float* ws = blk.ws + ((size_t)(b * blk.tiles + local) * H * kQT + r0 + rowa) * blk.ld + kc;
+  int st = 0, left = 0;                  // stage of the current key/value head, heads of its group still to come
+  for (int step = 0; step < steps; ++step) {
+    const int k0 = first + c0 + step * KW;
+    float s[HM][NB][4];
 #pragma unroll
-  for (int h = 0; h < HM; ++h) {
+    for (int h = 0; h < HM; h += R) {
 #pragma unroll
-    for (int n = 0; n < NB; ++n)
+      for (int r = 0; r < R; ++r)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) s[h][n][e] = 0.f;
-    if (h < p.H) {                       // block-uniform
-      if (h + 1 < p.H) {
-        fetch(h + 1);
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
-      } else {
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-      }
-      __syncthreads();
-      const bf16* qt = q_s + (h & 1) * kQT * dkp;
-      const bf16* kt = k_s + ((h / rep) & 1) * KW * dkp;
+        for (int n = 0; n < NB; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[h + r][n][e] = 0.f;
+      if (h < H) {                       // block-uniform
+        if (left == 0) {                 // a group begins: its keys are there, and the stage before may be filled again
+          if (stages == 3) asm volatile("cp.async.wait_group 1;" ::: "memory");
+          else asm volatile("cp.async.wait_group 0;" ::: "memory");
+          __syncthreads();
+          fetch();
+          left = rep;
+        }
+        left -= R;
+        const bf16* qt = q_s + h * kSq * dkp + (lane & 15) * dkp + (lane >> 4) * 8;
+        const bf16* kt = k_s + (st * KW + warp * 8 * NB) * dkp;
 #pragma unroll 4
-      for (int kk = 0; kk < dk16; kk += 16) {
-        uint32_t a[4];
-        ldsm_x4(a, qt + (wq * 16 + (lane & 15)) * dkp + kk + (lane >> 4) * 8);
-        if constexpr (NB >= 2) {
+        for (int kk = 0; kk < dk16; kk += 16) {
+          uint32_t a[R][4], bb[(NB + 1) / 2][4];
 #pragma unroll
-          for (int n = 0; n < NB; n += 2) {
-            uint32_t bb[4];
-            ldsm_x4(bb, kt + (wk * 8 * NB + n * 8 + (lane & 7) + ((lane >> 4) << 3)) * dkp + kk + ((lane >> 3) & 1) * 8);
-            mma_bf16(s[h][n], a, bb[0], bb[1]);
-            mma_bf16(s[h][n + 1], a, bb[2], bb[3]);
-          }
-        } else {                         // eight keys per warp: the other half of the load is not used
-          uint32_t bb[4];
-          ldsm_x4(bb, kt + (wk * 8 + (lane & 7)) * dkp + kk + ((lane >> 3) & 1) * 8);
-          mma_bf16(s[h][0], a, bb[0], bb[1]);
+          for (int r = 0; r < R; ++r) ldsm_x4(a[r], qt + r * kSq * dkp + kk);
+#pragma unroll
+          for (int n = 0; n < NB; n += 2)          // with eight keys per warp the other half of the load is not used
+            ldsm_x4(bb[n / 2], kt + (n * 8 + (lane & 7) + (NB > 1 ? (lane >> 4) << 3 : 0)) * dkp + kk + ((lane >> 3) & 1) * 8);
+#pragma unroll
+          for (int n = 0; n < NB; ++n)
+#pragma unroll
+            for (int r = 0; r < R; ++r) mma_bf16(s[h + r][n], a[r], bb[n / 2][(n & 1) * 2], bb[n / 2][(n & 1) * 2 + 1]);
+        }
+        if (left == 0 && ++st == stages) st = 0;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          // the distance is (r0 + row) - (k0 + key), from the step's smallest on
+          const float* pen = pen_s + (h + r) * kPen + rowa + KW - 1 - kc;
+#pragma unroll
+          for (int n = 0; n < NB; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+              const float x = s[h + r][n][e] * sx;
+              s[h + r][n][e] = (p.softcap > 0.f ? soft_cap_fast(x, cap2, p.softcap) : x) - pen[(e >> 1) * 8 - n * 8 - (e & 1)];
+            }
         }
       }
+    }
+    if (step + 1 < steps) {
+      __syncthreads();                   // nobody reads this step's penalties any more; the next group's barrier publishes the new ones
+      penalties(k0 + KW);
+    }
+    if (k0 - first + warp * 8 * NB < span) {       // mix and store; a tile's rows end with its span
+      bool seen[NB][4];
 #pragma unroll
       for (int n = 0; n < NB; ++n)
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-          // the distance is (q0 + row) - (k0 + key), from dmin on; rows past the portion's end stay inside the table
-          const float x = s[h][n][e] * sx, pen = pen_s[h * kPen + rowa + (e >> 1) * 8 + KW - 1 - (kc + n * 8 + (e & 1))];
-          s[h][n][e] = (p.softcap > 0.f ? soft_cap_fast(x, cap2, p.softcap) : x) - pen;
+          const int pos = k0 + kc + n * 8 + (e & 1), me = min(pa + (e >> 1) * 8, plast);
+          seen[n][e] = pos <= me && (p.window <= 0 || me - pos < p.window);
         }
-      __syncthreads();                   // before the stage is filled again
-    }
-  }
-  // mix and store
-  const int pa = p.pos0 + q0 + rowa;
-  float* ws = blk.ws + ((size_t)(b * blk.tiles + blockIdx.y) * p.H * kQT + rowa) * blk.ld + blockIdx.x * KW + kc;
-  for (int h = 0; h < p.H; ++h) {
-    float m[NB][4];
+      float* dst = ws + (k0 - first);
+      for (int h = 0; h < H; ++h) {
+        float m[NB][4];
 #pragma unroll
-    for (int n = 0; n < NB; ++n)
+        for (int n = 0; n < NB; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) m[n][e] = 0.f;
+          for (int e = 0; e < 4; ++e) m[n][e] = 0.f;
 #pragma unroll
-    for (int g = 0; g < HM; g += 2) {
-      const float2 t = *reinterpret_cast<const float2*>(talk_s + h * HM + g);
+        for (int g = 0; g < HM; g += 2) {
+          const float2 t = *reinterpret_cast<const float2*>(talk_s + h * HM + g);
 #pragma unroll
-      for (int n = 0; n < NB; ++n)
+          for (int n = 0; n < NB; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) m[n][e] = fmaf(t.x, s[g][n][e], fmaf(t.y, s[g + 1][n][e], m[n][e]));
-    }
+            for (int e = 0; e < 4; ++e) m[n][e] = fmaf(t.x, s[g][n][e], fmaf(t.y, s[g + 1][n][e], m[n][e]));
+        }
 #pragma unroll
-    for (int n = 0; n < NB; ++n) {
-      float r[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int pos = k0 + kc + n * 8 + (e & 1), me = min(pa + (e >> 1) * 8, p.pos0 + p.T - 1);
-        r[e] = pos <= me && (p.window <= 0 || me - pos < p.window) ? m[n][e] : -INFINITY;
+        for (int n = 0; n < NB; ++n) {
+          *reinterpret_cast<float2*>(dst + n * 8) = make_float2(seen[n][0] ? m[n][0] : -INFINITY, seen[n][1] ? m[n][1] : -INFINITY);
+          *reinterpret_cast<float2*>(dst + (size_t)8 * blk.ld + n * 8) = make_float2(seen[n][2] ? m[n][2] : -INFINITY, seen[n][3] ? m[n][3] : -INFINITY);
+        }
+        dst += (size_t)kQT * blk.ld;
       }
-      *reinterpret_cast<float2*>(ws + (size_t)h * kQT * blk.ld + n * 8) = make_float2(r[0], r[1]);
-      *reinterpret_cast<float2*>(ws + ((size_t)h * kQT + 8) * blk.ld + n * 8) = make_float2(r[2], r[3]);
     }
   }
 }
@@ -239,7 +266,7 @@ template <typename T> __global__ void __launch_bounds__(256) talk_scores_kernel(
 constexpr int kPvThreads = 128;
 
 template <int VD>
-__global__ void __launch_bounds__(kPvThreads) talk_values_bf16_kernel(const nb_talk_attention_args p, TalkBlock blk, int vtiles, int vec) {
+__global__ void __launch_bounds__(kPvThreads, VD <= 128 ? 3 : 1) talk_values_bf16_kernel(const nb_talk_attention_args p, TalkBlock blk, int vtiles, int vec) {
   extern __shared__ __align__(16) bf16 v_s[];   // [2][64][VD + 8]
   constexpr int vp = VD + 8;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -727,19 +754,36 @@ static int talk_ld(int T, int pos0, int window) {      // longest span of a quer
   return (int)((span + kKT - 1) / kKT * kKT);
 }
 
-template <int HM, int NB> static int launch_scores_bf16(const nb_talk_attention_args& a, const TalkBlock& blk, cudaStream_t st) {
-  const int dk16 = (a.dim + 15) & ~15, KW = 16 * NB;
-  const size_t smem = (size_t)2 * (kQT + KW) * (dk16 + 8) * 2 + ((size_t)a.H * HM + (size_t)a.H * (kQT + KW)) * 4;
+constexpr size_t kTalkSmem = 220 * 1024;
+
+static size_t talk_scores_smem(const nb_talk_attention_args& a, int HM, int NB, int stages) {
+  const int dkp = ((a.dim + 15) & ~15) + 8, KW = 64 * NB;
+  return (size_t)(a.H * kSq + stages * KW) * dkp * 2 + ((size_t)a.H * HM + (size_t)a.H * (kSq + KW)) * 4;
+}
+
+template <int HM, int NB, bool kTwo> static int launch_scores_mma(const nb_talk_attention_args& a, const TalkBlock& blk, int stages, cudaStream_t st) {
   static bool done[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (!done[dev & 63]) {
-    if (cudaError_t e = cudaFuncSetAttribute(talk_scores_bf16_kernel<HM, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)) return record_cuda_error(e);
+    if (cudaError_t e = cudaFuncSetAttribute(talk_scores_bf16_kernel<HM, NB, kTwo>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kTalkSmem))
+      return record_cuda_error(e);
     done[dev & 63] = true;
   }
   const int vec = a.dim % 8 == 0 && a.ldq % 8 == 0 && a.ldc % 8 == 0 && (uintptr_t)a.q % 16 == 0 && (uintptr_t)a.cache % 16 == 0;
-  talk_scores_bf16_kernel<HM, NB><<<dim3(blk.ld / KW, blk.tiles, a.B), kScThreads, smem, st>>>(a, blk, dk16, vec);
+  const int steps = (blk.ld + 64 * NB - 1) / (64 * NB), subs = blk.tiles * (kQT / kSq);
+  const int chunk = std::max(1, std::min(steps, (int)((long long)steps * subs * a.B / (4 * sm_count()))));   // about four CTAs per SM
+  talk_scores_bf16_kernel<HM, NB, kTwo><<<dim3((steps + chunk - 1) / chunk, subs, a.B), kScThreads, talk_scores_smem(a, HM, NB, stages), st>>>(
+      a, blk, (a.dim + 15) & ~15, chunk, stages, vec);
   return check_launch();
+}
+
+// Whether the tensor-core kernel takes the sizes; launches it if so (rc: its status).
+template <int HM, int NB> static bool launch_scores_bf16(const nb_talk_attention_args& a, const TalkBlock& blk, cudaStream_t st, int& rc) {
+  const int stages = talk_scores_smem(a, HM, NB, 3) <= kTalkSmem ? 3 : 2;
+  if (a.H > HM || talk_scores_smem(a, HM, NB, stages) > kTalkSmem) return false;
+  rc = (a.H / a.G) % 2 == 0 ? launch_scores_mma<HM, NB, true>(a, blk, stages, st) : launch_scores_mma<HM, NB, false>(a, blk, stages, st);
+  return true;
 }
 
 template <typename T> static int launch_scores_simple(const nb_talk_attention_args& a, const TalkBlock& blk, cudaStream_t st) {
@@ -818,26 +862,20 @@ extern "C" int nb_talk_attention(const nb_talk_attention_args* a, void* workspac
   cudaStream_t st = (cudaStream_t)stream;
   const int all = (a->T + kQT - 1) / kQT, fit = std::min<size_t>(std::min<size_t>(workspace_bytes / one, all), 16000 / a->B + 1);
   const int blocks = (all + fit - 1) / fit, per = (all + blocks - 1) / blocks;     // equal blocks
-  const int dk16 = (a->dim + 15) & ~15;
-  const bool mma = a->dtype == NB_BF16 && a->H <= 40 && (size_t)2 * 128 * (dk16 + 8) * 2 + (size_t)a->H * 200 * 4 <= 200 * 1024;
   for (int t = 0; t < all; t += per) {
     TalkBlock blk;
     blk.ws = reinterpret_cast<float*>(workspace);
     blk.tile0 = t;
     blk.tiles = std::min(per, all - t);
     blk.ld = talk_ld(a->T, a->pos0, a->window);
-    int rc;
-    if (mma) {
-      rc = a->H <= 4    ? launch_scores_bf16<4, 4>(*a, blk, st)
-           : a->H <= 6  ? launch_scores_bf16<6, 4>(*a, blk, st)
-           : a->H <= 8  ? launch_scores_bf16<8, 4>(*a, blk, st)
-           : a->H <= 10 ? launch_scores_bf16<10, 4>(*a, blk, st)
-           : a->H <= 16 ? launch_scores_bf16<16, 2>(*a, blk, st)
-           : a->H <= 20 ? launch_scores_bf16<20, 2>(*a, blk, st)
-           : a->H <= 32 ? launch_scores_bf16<32, 1>(*a, blk, st)
-                        : launch_scores_bf16<40, 1>(*a, blk, st);
+    int rc = NB_OK;
+    if (a->dtype == NB_F32) {
+      rc = launch_scores_simple<float>(*a, blk, st);
     } else {
-      rc = a->dtype == NB_F32 ? launch_scores_simple<float>(*a, blk, st) : launch_scores_simple<bf16>(*a, blk, st);
+      const bool taken = (blk.ld > 256 && launch_scores_bf16<10, 4>(*a, blk, st, rc)) || launch_scores_bf16<10, 2>(*a, blk, st, rc) ||
+                         (blk.ld > 64 && launch_scores_bf16<20, 2>(*a, blk, st, rc)) || launch_scores_bf16<20, 1>(*a, blk, st, rc) ||
+                         launch_scores_bf16<40, 1>(*a, blk, st, rc);
+      if (!taken) rc = launch_scores_simple<bf16>(*a, blk, st);
     }
     if (rc) return rc;
     if (a->dtype == NB_BF16)
