@@ -492,7 +492,7 @@ __host__ __device__ inline int head_row(int H) { return pad4(H) | 4; }
 struct TalkDecodeSmem {                  // float offsets; the staged rows follow at `rows`
   int q, talk, sc, mx, acc, ml, xch, xml, wr, rows, dimp, hp, per, slot;
   __host__ __device__ TalkDecodeSmem(const nb_talk_decode_args& a, int S, int stage) {
-    dimp = pad4(a.dim);
+    dimp = (a.dim + 15) & ~15;
     hp = head_row(a.H);
     per = pad4((a.H * a.vdim + S - 1) / S);
     slot = per;
@@ -580,10 +580,8 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
 
   pdl_enter();
   const float* row = p.p + (size_t)b * p.ldp;
-  for (int i = tid; i < H * L.dimp; i += kTdThreads) {
-    const int h = i / L.dimp, d = i - h * L.dimp;
-    qs[i] = d < D ? row[p.q_off + h * D + d] : 0.f;
-  }
+  for (int h = warp; h < H; h += kTdWarps)
+    for (int d = lane; d < L.dimp; d += 32) qs[h * L.dimp + d] = d < D ? row[p.q_off + h * D + d] : 0.f;
   auto put_row = [&](T* dst) {           // this position's keys and values: staged, and into the cache
     T* crow = cache + (size_t)pos * p.ldc;
     for (int i = tid; i < p.ldc; i += kTdThreads) {
@@ -593,7 +591,7 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
       crow[i] = v;
     }
   };
-  const bool dvec = D % 8 == 0, vvec = V % 2 == 0;
+  const bool dvec = D % 8 == 0, vvec = V % 2 == 0, mma = sizeof(T) == 2 && D % 8 == 0 && V % 8 == 0;
   const float isc = p.softcap > 0.f ? p.scale / p.softcap : p.scale;
   for (int base = 0; base < cnt; base += stage) {
     const int nk = min(stage, cnt - base);
@@ -605,55 +603,91 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     if (mine >= base && mine < base + nk) put_row(rows + (size_t)(mine - base) * ldr);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    // raw scores: a thread takes one key of one group (and up to four of its heads at a time)
-    const int chunks = (rep + 3) / 4;
-    for (int i = tid; i < nk * p.G * chunks; i += kTdThreads) {
-      const int gc = i / nk, j = i - gc * nk, g = gc / chunks, h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
-      const T* kr = rows + (size_t)j * ldr + g * D;
-      const float* qh = qs + h0 * L.dimp;
-      float x[4] = {0.f, 0.f, 0.f, 0.f};
-      if (dvec) {
-        for (int d = 0; d < D; d += 8) {
-          float kv[8];
-          load8(kr + d, kv);
+    const int chunks = (rep + 3) / 4, tiles16 = (rep + 15) / 16;
+    auto put_score = [&](int j, int h, float x) {                  // over the penalty that waits there
+      float* s = sc + j * hp + h;
+      *s = (p.softcap > 0.f ? p.softcap * tanhf(x * isc) : x * isc) - *s;
+    };
+    const int ra = lane >> 2, c2 = (lane & 3) * 2;                 // this lane's first row (head) and column pair of a product
+    if (mma) {
+      // raw scores on the tensor cores: up to 16 heads of a group x 16 keys per warp; the queries enter as three bf16 terms (a score's
+      // error is an exponent's)
+      const int kt = (nk + 15) / 16;
+      for (int i = warp; i < p.G * tiles16 * kt; i += kTdWarps) {
+        const int gc = i / kt, j0 = (i - gc * kt) * 16, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
+        const bf16* kr = reinterpret_cast<const bf16*>(rows) + (size_t)min(j0 + (lane & 7) + ((lane >> 4) << 3), nk - 1) * ldr + g * D + ((lane >> 3) & 1) * 8;
+        float c[2][4] = {};
+        for (int kk = 0; kk < D; kk += 16) {
+          uint32_t q1[4], q2[4], q3[4], bb[4];
+          ldsm_x4(bb, kr + kk);
 #pragma unroll
-          for (int r = 0; r < 4; ++r)
-            if (r < hn) {
-              const float4 a = *reinterpret_cast<const float4*>(qh + r * L.dimp + d), c = *reinterpret_cast<const float4*>(qh + r * L.dimp + d + 4);
-              x[r] += (kv[0] * a.x + kv[1] * a.y) + (kv[2] * a.z + kv[3] * a.w) + ((kv[4] * c.x + kv[5] * c.y) + (kv[6] * c.z + kv[7] * c.w));
-            }
+          for (int f = 0; f < 4; ++f) {
+            const int r = ra + (f & 1) * 8;
+            const float2 v = r < hn ? *reinterpret_cast<const float2*>(qs + (hb + r) * L.dimp + kk + (f >> 1) * 8 + c2) : make_float2(0.f, 0.f);
+            split_bf16(v.x, v.y, q1[f], q2[f]);
+            q3[f] = pack_bf16(v.x - bf_lo(q1[f]) - bf_lo(q2[f]), v.y - bf_hi(q1[f]) - bf_hi(q2[f]));
+          }
+          mma_bf16(c[0], q1, bb[0], bb[1]);
+          mma_bf16(c[1], q1, bb[2], bb[3]);
+          mma_bf16(c[0], q2, bb[0], bb[1]);
+          mma_bf16(c[1], q2, bb[2], bb[3]);
+          mma_bf16(c[0], q3, bb[0], bb[1]);
+          mma_bf16(c[1], q3, bb[2], bb[3]);
         }
-      } else {
-        for (int d = 0; d < D; ++d) {
-          const float kv = to_f(kr[d]);
 #pragma unroll
-          for (int r = 0; r < 4; ++r)
-            if (r < hn) x[r] = fmaf(kv, qh[r * L.dimp + d], x[r]);
-        }
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int j = j0 + x * 8 + c2 + (e & 1), r = ra + (e >> 1) * 8;
+            if (j < nk && r < hn) put_score(j, hb + r, c[x][e]);
+          }
       }
+    } else {
+      // a thread takes one key of one group (and up to four of its heads at a time)
+      for (int i = tid; i < nk * p.G * chunks; i += kTdThreads) {
+        const int gc = i / nk, j = i - gc * nk, g = gc / chunks, h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
+        const T* kr = rows + (size_t)j * ldr + g * D;
+        const float* qh = qs + h0 * L.dimp;
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (dvec) {
+          for (int d = 0; d < D; d += 8) {
+            float kv[8];
+            load8(kr + d, kv);
 #pragma unroll
-      for (int r = 0; r < 4; ++r)
-        if (r < hn) {
-          float* s = sc + j * hp + h0 + r;
-          *s = (p.softcap > 0.f ? p.softcap * tanhf(x[r] * isc) : x[r] * isc) - *s;
+            for (int r = 0; r < 4; ++r)
+              if (r < hn) {
+                const float4 a = *reinterpret_cast<const float4*>(qh + r * L.dimp + d), c = *reinterpret_cast<const float4*>(qh + r * L.dimp + d + 4);
+                x[r] += (kv[0] * a.x + kv[1] * a.y) + (kv[2] * a.z + kv[3] * a.w) + ((kv[4] * c.x + kv[5] * c.y) + (kv[6] * c.z + kv[7] * c.w));
+              }
+          }
+        } else {
+          for (int d = 0; d < D; ++d) {
+            const float kv = to_f(kr[d]);
+#pragma unroll
+            for (int r = 0; r < 4; ++r)
+              if (r < hn) x[r] = fmaf(kv, qh[r * L.dimp + d], x[r]);
+          }
         }
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+          if (r < hn) put_score(j, h0 + r, x[r]);
+      }
     }
     __syncthreads();
-    for (int i = tid; i < nk * H; i += kTdThreads) {               // mixed scores
-      const int h = i / nk, j = i - h * nk;
-      const float *t = talk_s + h * hp, *s = sc + j * hp;
-      float m = 0.f;
-      for (int g = 0; g < hp; g += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(t + g), c = *reinterpret_cast<const float4*>(s + g);
-        m = fmaf(a.x, c.x, m); m = fmaf(a.y, c.y, m); m = fmaf(a.z, c.z, m); m = fmaf(a.w, c.w, m);
+    // mixed scores and the running softmax, a warp per head
+    for (int h = warp; h < H; h += kTdWarps) {
+      const float *t = talk_s + h * hp, old = ml[h];
+      float m = old;
+      for (int j = lane; j < nk; j += 32) {
+        const float* s = sc + j * hp;
+        float v = 0.f;
+        for (int g = 0; g < hp; g += 4) {
+          const float4 a = *reinterpret_cast<const float4*>(t + g), c = *reinterpret_cast<const float4*>(s + g);
+          v = fmaf(a.x, c.x, v); v = fmaf(a.y, c.y, v); v = fmaf(a.z, c.z, v); v = fmaf(a.w, c.w, v);
+        }
+        mx[j * hp + h] = v;
+        m = fmaxf(m, v);
       }
-      mx[j * hp + h] = m;
-    }
-    __syncthreads();
-    for (int h = warp; h < H; h += kTdWarps) {                     // running softmax, a warp per head
-      float m = ml[h];
-      const float old = m;
-      for (int j = lane; j < nk; j += 32) m = fmaxf(m, mx[j * hp + h]);
       m = warp_max(m);
       float sum = 0.f;
       for (int j = lane; j < nk; j += 32) {
@@ -670,39 +704,73 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
       }
     }
     __syncthreads();
-    // weighted values: a thread takes two columns (one if their number is odd) of up to four heads of a group
-    const int vw = vvec ? 2 : 1, cols = V / vw;
-    for (int i = tid; i < p.G * chunks * cols; i += kTdThreads) {
-      const int gc = i / cols, c = (i - gc * cols) * vw, g = gc / chunks, h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
-      const T* vr = rows + p.v_off + g * V + c;
-      float2 o[4] = {};
-      if (vvec) {
-#pragma unroll 4
-        for (int j = 0; j < nk; ++j) {
-          const float2 v = load2(vr + (size_t)j * ldr);
+    if (mma) {
+      // weighted values: up to 16 heads of a group x 16 columns per warp; the weights enter as two bf16 terms
+      const int ct = (V + 15) / 16;
+      for (int i = warp; i < p.G * tiles16 * ct; i += kTdWarps) {
+        const int gc = i / ct, v0 = (i - gc * ct) * 16, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
+        const bf16* vr = reinterpret_cast<const bf16*>(rows) + p.v_off + g * V + v0 + (lane >> 4) * 8;
+        float c[2][4] = {};
+        for (int kk = 0; kk < nk; kk += 16) {
+          uint32_t hi[4], lo[4], bb[4];
+          ldsm_x4_t(bb, vr + (size_t)min(kk + (lane & 15), nk - 1) * ldr);         // keys past the stage have no weight
 #pragma unroll
-          for (int r = 0; r < 4; ++r)
-            if (r < hn) {
-              const float w = mx[j * hp + h0 + r];
-              o[r].x = fmaf(w, v.x, o[r].x);
-              o[r].y = fmaf(w, v.y, o[r].y);
+          for (int f = 0; f < 4; ++f) {
+            const int r = ra + (f & 1) * 8, j = kk + (f >> 1) * 8 + c2;
+            const float* w = mx + j * hp + hb + r;
+            split_bf16(r < hn && j < nk ? w[0] : 0.f, r < hn && j + 1 < nk ? w[hp] : 0.f, hi[f], lo[f]);
+          }
+          mma_bf16(c[0], hi, bb[0], bb[1]);
+          mma_bf16(c[1], hi, bb[2], bb[3]);
+          mma_bf16(c[0], lo, bb[0], bb[1]);
+          mma_bf16(c[1], lo, bb[2], bb[3]);
+        }
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int v = v0 + x * 8 + c2 + (e & 1), r = ra + (e >> 1) * 8;
+            if (v < V && r < hn) {
+              float* a = acc + (hb + r) * V + v;
+              *a = *a * wr[hb + r] + c[x][e];
             }
-        }
-      } else {
-        for (int j = 0; j < nk; ++j) {
-          const float v = to_f(vr[(size_t)j * ldr]);
-#pragma unroll
-          for (int r = 0; r < 4; ++r)
-            if (r < hn) o[r].x = fmaf(mx[j * hp + h0 + r], v, o[r].x);
-        }
+          }
       }
+    } else {
+      // a thread takes two columns (one if their number is odd) of up to four heads of a group
+      const int vw = vvec ? 2 : 1, cols = V / vw;
+      for (int i = tid; i < p.G * chunks * cols; i += kTdThreads) {
+        const int gc = i / cols, c = (i - gc * cols) * vw, g = gc / chunks, h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
+        const T* vr = rows + p.v_off + g * V + c;
+        float2 o[4] = {};
+        if (vvec) {
+#pragma unroll 4
+          for (int j = 0; j < nk; ++j) {
+            const float2 v = load2(vr + (size_t)j * ldr);
 #pragma unroll
-      for (int r = 0; r < 4; ++r)
-        if (r < hn) {
-          float* a = acc + (h0 + r) * V + c;
-          a[0] = a[0] * wr[h0 + r] + o[r].x;
-          if (vvec) a[1] = a[1] * wr[h0 + r] + o[r].y;
+            for (int r = 0; r < 4; ++r)
+              if (r < hn) {
+                const float w = mx[j * hp + h0 + r];
+                o[r].x = fmaf(w, v.x, o[r].x);
+                o[r].y = fmaf(w, v.y, o[r].y);
+              }
+          }
+        } else {
+          for (int j = 0; j < nk; ++j) {
+            const float v = to_f(vr[(size_t)j * ldr]);
+#pragma unroll
+            for (int r = 0; r < 4; ++r)
+              if (r < hn) o[r].x = fmaf(mx[j * hp + h0 + r], v, o[r].x);
+          }
         }
+#pragma unroll
+        for (int r = 0; r < 4; ++r)
+          if (r < hn) {
+            float* a = acc + (h0 + r) * V + c;
+            a[0] = a[0] * wr[h0 + r] + o[r].x;
+            if (vvec) a[1] = a[1] * wr[h0 + r] + o[r].y;
+          }
+      }
     }
   }
   __syncthreads();
@@ -726,15 +794,11 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     gate[u] = p.g_off >= 0 && i < sn ? row[p.g_off + s0 + i] : 0.f;
   }
   cluster.sync();                        // nobody touches another CTA's shared memory after this
-  for (int h = tid; h < H; h += kTdThreads) {
-    float m = -FLT_MAX, den = 0.f;
-    for (int r = 0; r < S; ++r) m = fmaxf(m, xml[r * 2 * hp + h]);
-    for (int r = 0; r < S; ++r) {        // a CTA without keys has maximum -FLT_MAX and sum 0
-      const float w = expf(xml[r * 2 * hp + h] - m);
-      wr[r * hp + h] = w;
-      den += w * xml[r * 2 * hp + hp + h];
-    }
-    wr[S * hp + h] = 1.f / den;
+  for (int h = warp; h < H; h += kTdWarps) {       // a CTA without keys has maximum -FLT_MAX and sum 0
+    const float mr = lane < S ? xml[lane * 2 * hp + h] : -FLT_MAX, w = expf(mr - warp_max(mr));
+    const float den = warp_sum(lane < S ? w * xml[lane * 2 * hp + hp + h] : 0.f);
+    if (lane < S) wr[lane * hp + h] = w;
+    if (lane == 0) wr[S * hp + h] = 1.f / den;
   }
   __syncthreads();
   for (int i = tid, u = 0; i < sn; i += kTdThreads, ++u) {
@@ -922,12 +986,12 @@ template <typename T> static int launch_talk_decode(const nb_talk_decode_args& a
   int S = 1;
   while (S < widest[dev & 63] && S * 8 < most && a.B * S * 2 <= 256) S *= 2;
   const size_t row = (size_t)((a.ldc * sizeof(T) / 16) | 1) * 16, per_key = row + (size_t)2 * head_row(a.H) * 4;
-  const size_t fixed = (size_t)TalkDecodeSmem(a, S, 0).rows * 4;
+  const size_t fixed = (size_t)TalkDecodeSmem(a, S, 0).rows * 4 + 32;
   if (fixed + per_key > kMax) return NB_ERR_SHAPE;
   const int stage = (int)std::min<size_t>((most + S - 1) / S, (kMax - fixed) / per_key);
   attr[0].val.clusterDim.z = S;
   cfg.gridDim = dim3(1, a.B, S);
-  cfg.dynamicSmemBytes = (size_t)TalkDecodeSmem(a, S, stage).rows * 4 + stage * row;
+  cfg.dynamicSmemBytes = (size_t)TalkDecodeSmem(a, S, stage).rows * 4 + stage * row + 32;   // 16-column reads of the last row
   cfg.numAttrs = 2;
   return record_cuda_error(cudaLaunchKernelEx(&cfg, kernel, a, stage));
 }

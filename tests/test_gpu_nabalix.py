@@ -263,7 +263,7 @@ def test_talk_decode(dev, shape, dtype, pos, window):
     L.talk_decode(p=p.data_ptr(), cache=cache.data_ptr(), penalty=pen.data_ptr(), talk=tk.data_ptr(), pos=pt.data_ptr(), out=out.data_ptr(), scale=scale,
                   softcap=cap, cache_dtype=L._DTYPE[dtype], B=B, H=H, G=G, dim=D, vdim=V, ctx=ctx, ldc=cache.shape[2], v_off=v_off, ldp=p.shape[1],
                   q_off=0, k_off=k_off, g_off=g_off, ldo=H * V, window=window, n_pen=n_pen)
-    close(out, ref, 2e-5)
+    close(out, ref, 2e-5 if dtype == F32 else 5e-5)                 # bf16: softmax weights as two bf16 terms
     assert torch.equal(cache[:, pos], want_row) and cache[:, N:].isnan().all()
 
 
