@@ -482,7 +482,7 @@ __global__ void __launch_bounds__(128) talk_values_kernel(const nb_talk_attentio
 // running maximum and sum per head; then every CTA sends its weighted values in slices to the CTAs that merge them.  Rows
 // of earlier positions, the talk matrix and the penalties do not depend on the launch before: they are requested ahead of
 // the dependency wait.
-constexpr int kTdThreads = 512, kTdWarps = kTdThreads / 32;
+constexpr int kTdThreads = 640, kTdWarps = kTdThreads / 32;
 
 __host__ __device__ inline int pad4(int n) { return (n + 3) & ~3; }
 // row length of a table [key][head]: a multiple of 4 that is odd in units of 4, so that 16-byte reads of neighbouring keys
@@ -574,22 +574,37 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     sc[j * hp + c] = mx[j * hp + c] = 0.f;
   }
   penalties(0, min(stage, cnt));
-  for (int i = tid; i < H * V; i += kTdThreads) acc[i] = 0.f;
+  for (int i = tid; i < pad4(H * V); i += kTdThreads) acc[i] = 0.f;
   for (int i = tid; i < hp; i += kTdThreads) { ml[i] = -FLT_MAX; ml[hp + i] = 0.f; }
   cluster.barrier_arrive();
 
   pdl_enter();
   const float* row = p.p + (size_t)b * p.ldp;
+  auto row_value = [&](int i) {          // element i of this position's row
+    const bool in = i < p.G * D || (i >= p.v_off && i < p.v_off + p.G * V);
+    return in ? row[p.k_off + i] : 0.f;
+  };
+  constexpr int kRowPre = 4;             // elements of it per thread that are requested with the queries
+  float rv[kRowPre];
+  if (mine >= 0 && mine < cnt) {
+#pragma unroll
+    for (int u = 0; u < kRowPre; ++u) rv[u] = tid + u * kTdThreads < p.ldc ? row_value(tid + u * kTdThreads) : 0.f;
+  }
+#pragma unroll 4
   for (int h = warp; h < H; h += kTdWarps)
+#pragma unroll 4
     for (int d = lane; d < L.dimp; d += 32) qs[h * L.dimp + d] = d < D ? row[p.q_off + h * D + d] : 0.f;
   auto put_row = [&](T* dst) {           // this position's keys and values: staged, and into the cache
     T* crow = cache + (size_t)pos * p.ldc;
-    for (int i = tid; i < p.ldc; i += kTdThreads) {
-      const bool in = i < p.G * D || (i >= p.v_off && i < p.v_off + p.G * V);
-      const T v = from_f<T>(in ? row[p.k_off + i] : 0.f);
+    auto put = [&](int i, float x) {
+      const T v = from_f<T>(x);
       dst[i] = v;
       crow[i] = v;
-    }
+    };
+#pragma unroll
+    for (int u = 0; u < kRowPre; ++u)
+      if (tid + u * kTdThreads < p.ldc) put(tid + u * kTdThreads, rv[u]);
+    for (int i = tid + kRowPre * kTdThreads; i < p.ldc; i += kTdThreads) put(i, row_value(i));
   };
   const bool dvec = D % 8 == 0, vvec = V % 2 == 0, mma = sizeof(T) == 2 && D % 8 == 0 && V % 8 == 0;
   const float isc = p.softcap > 0.f ? p.scale / p.softcap : p.scale;
@@ -616,7 +631,8 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
       for (int i = warp; i < p.G * tiles16 * kt; i += kTdWarps) {
         const int gc = i / kt, j0 = (i - gc * kt) * 16, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
         const bf16* kr = reinterpret_cast<const bf16*>(rows) + (size_t)min(j0 + (lane & 7) + ((lane >> 4) << 3), nk - 1) * ldr + g * D + ((lane >> 3) & 1) * 8;
-        float c[2][4] = {};
+        float c[3][2][4] = {};           // a chain of products per term
+#pragma unroll 4
         for (int kk = 0; kk < D; kk += 16) {
           uint32_t q1[4], q2[4], q3[4], bb[4];
           ldsm_x4(bb, kr + kk);
@@ -627,20 +643,30 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
             split_bf16(v.x, v.y, q1[f], q2[f]);
             q3[f] = pack_bf16(v.x - bf_lo(q1[f]) - bf_lo(q2[f]), v.y - bf_hi(q1[f]) - bf_hi(q2[f]));
           }
-          mma_bf16(c[0], q1, bb[0], bb[1]);
-          mma_bf16(c[1], q1, bb[2], bb[3]);
-          mma_bf16(c[0], q2, bb[0], bb[1]);
-          mma_bf16(c[1], q2, bb[2], bb[3]);
-          mma_bf16(c[0], q3, bb[0], bb[1]);
-          mma_bf16(c[1], q3, bb[2], bb[3]);
+          mma_bf16(c[0][0], q1, bb[0], bb[1]);
+          mma_bf16(c[0][1], q1, bb[2], bb[3]);
+          mma_bf16(c[1][0], q2, bb[0], bb[1]);
+          mma_bf16(c[1][1], q2, bb[2], bb[3]);
+          mma_bf16(c[2][0], q3, bb[0], bb[1]);
+          mma_bf16(c[2][1], q3, bb[2], bb[3]);
         }
 #pragma unroll
-        for (int x = 0; x < 2; ++x)
+        for (int half = 0; half < 2; ++half) {
+          if (half * 8 >= hn) break;
+          const int r = ra + half * 8;
+          float v[4];
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
-            const int j = j0 + x * 8 + c2 + (e & 1), r = ra + (e >> 1) * 8;
-            if (j < nk && r < hn) put_score(j, hb + r, c[x][e]);
+            const float x = ((c[2][e >> 1][2 * half + (e & 1)] + c[1][e >> 1][2 * half + (e & 1)]) + c[0][e >> 1][2 * half + (e & 1)]) * isc;
+            // cap tanh(x) = cap - 2 cap / (1 + e^2x): an absolute error of the cap's rounding
+            v[e] = p.softcap > 0.f ? p.softcap - 2.f * p.softcap / (1.f + expf(2.f * x)) : x;
           }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int j = j0 + (e >> 1) * 8 + c2 + (e & 1);
+            if (j < nk && r < hn) sc[j * hp + hb + r] = v[e] - sc[j * hp + hb + r];
+          }
+        }
       }
     } else {
       // a thread takes one key of one group (and up to four of its heads at a time)
@@ -681,9 +707,10 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
       for (int j = lane; j < nk; j += 32) {
         const float* s = sc + j * hp;
         float v = 0.f;
+#pragma unroll 4
         for (int g = 0; g < hp; g += 4) {
           const float4 a = *reinterpret_cast<const float4*>(t + g), c = *reinterpret_cast<const float4*>(s + g);
-          v = fmaf(a.x, c.x, v); v = fmaf(a.y, c.y, v); v = fmaf(a.z, c.z, v); v = fmaf(a.w, c.w, v);
+          v += (a.x * c.x + a.y * c.y) + (a.z * c.z + a.w * c.w);
         }
         mx[j * hp + h] = v;
         m = fmaxf(m, v);
@@ -705,35 +732,51 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     }
     __syncthreads();
     if (mma) {
-      // weighted values: up to 16 heads of a group x 16 columns per warp; the weights enter as two bf16 terms
-      const int ct = (V + 15) / 16;
-      for (int i = warp; i < p.G * tiles16 * ct; i += kTdWarps) {
-        const int gc = i / ct, v0 = (i - gc * ct) * 16, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
-        const bf16* vr = reinterpret_cast<const bf16*>(rows) + p.v_off + g * V + v0 + (lane >> 4) * 8;
-        float c[2][4] = {};
+      // weighted values: up to 16 heads of a group x up to kCt tiles of 16 columns per warp; the weights enter as two bf16 terms
+      constexpr int kCt = 4;
+      const int ct = (V + 15) / 16, tpw = min(kCt, (p.G * tiles16 * ct + kTdWarps - 1) / kTdWarps), parts = (ct + tpw - 1) / tpw;
+      for (int i = warp; i < p.G * tiles16 * parts; i += kTdWarps) {
+        const int gc = i / parts, t0 = (i - gc * parts) * tpw, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
+        const int tn = min(tpw, ct - t0);
+        const bf16* vr = reinterpret_cast<const bf16*>(rows) + p.v_off + g * V + t0 * 16 + (lane >> 4) * 8;
+        float c[kCt][2][4] = {};
+#pragma unroll 2
         for (int kk = 0; kk < nk; kk += 16) {
-          uint32_t hi[4], lo[4], bb[4];
-          ldsm_x4_t(bb, vr + (size_t)min(kk + (lane & 15), nk - 1) * ldr);         // keys past the stage have no weight
+          uint32_t hi[4], lo[4];
 #pragma unroll
           for (int f = 0; f < 4; ++f) {
             const int r = ra + (f & 1) * 8, j = kk + (f >> 1) * 8 + c2;
             const float* w = mx + j * hp + hb + r;
             split_bf16(r < hn && j < nk ? w[0] : 0.f, r < hn && j + 1 < nk ? w[hp] : 0.f, hi[f], lo[f]);
           }
-          mma_bf16(c[0], hi, bb[0], bb[1]);
-          mma_bf16(c[1], hi, bb[2], bb[3]);
-          mma_bf16(c[0], lo, bb[0], bb[1]);
-          mma_bf16(c[1], lo, bb[2], bb[3]);
+          const bf16* vk = vr + (size_t)min(kk + (lane & 15), nk - 1) * ldr;       // keys past the stage have no weight
+          uint32_t bb[kCt][4];
+#pragma unroll
+          for (int y = 0; y < kCt; ++y)
+            if (y < tn) ldsm_x4_t(bb[y], vk + y * 16);
+#pragma unroll
+          for (int term = 0; term < 2; ++term)
+#pragma unroll
+            for (int y = 0; y < kCt; ++y)
+              if (y < tn) {
+                mma_bf16(c[y][0], term ? lo : hi, bb[y][0], bb[y][1]);
+                mma_bf16(c[y][1], term ? lo : hi, bb[y][2], bb[y][3]);
+              }
         }
 #pragma unroll
-        for (int x = 0; x < 2; ++x)
+        for (int y = 0; y < kCt; ++y)
+          if (y < tn) {
 #pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int v = v0 + x * 8 + c2 + (e & 1), r = ra + (e >> 1) * 8;
-            if (v < V && r < hn) {
-              float* a = acc + (hb + r) * V + v;
-              *a = *a * wr[hb + r] + c[x][e];
-            }
+            for (int x = 0; x < 2; ++x)
+#pragma unroll
+              for (int half = 0; half < 2; ++half) {
+                const int v = (t0 + y) * 16 + x * 8 + c2, r = ra + half * 8;       // V is a multiple of 8
+                if (v < V && r < hn) {
+                  float2* a = reinterpret_cast<float2*>(acc + (hb + r) * V + v);
+                  const float f = wr[hb + r];
+                  *a = make_float2(fmaf(a->x, f, c[y][x][2 * half]), fmaf(a->y, f, c[y][x][2 * half + 1]));
+                }
+              }
           }
       }
     } else {
@@ -776,13 +819,12 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
   __syncthreads();
   cluster.barrier_wait();                // every CTA of the cluster runs: its shared memory may be written from here on
   const int HV = H * V;
-  for (int i = tid; i < HV; i += kTdThreads) {
-    const int to = i / L.per;
-    cluster.map_shared_rank(xch, to)[rank * L.slot + i - to * L.per] = acc[i];
-  }
-  for (int i = tid; i < 2 * hp * S; i += kTdThreads) {
-    const int to = i / (2 * hp), c = i - to * 2 * hp;
-    cluster.map_shared_rank(xml, to)[rank * 2 * hp + c] = ml[c];
+  for (int to = warp; to < S; to += kTdWarps) {  // slices, maxima and sums in fours; acc is padded to them
+    float4* x = reinterpret_cast<float4*>(cluster.map_shared_rank(xch, to) + rank * L.slot);
+    const float4* a = reinterpret_cast<const float4*>(acc + to * L.per);
+    for (int i = lane; i < min(L.per, HV - to * L.per + 3) / 4; i += 32) x[i] = a[i];
+    float4* y = reinterpret_cast<float4*>(cluster.map_shared_rank(xml, to) + rank * 2 * hp);
+    for (int i = lane; i < hp / 2; i += 32) y[i] = reinterpret_cast<const float4*>(ml)[i];
   }
   // the gate of this CTA's slice travels meanwhile
   const int s0 = rank * L.per, sn = max(0, min(L.per, HV - s0));
