@@ -492,7 +492,7 @@ __host__ __device__ inline int head_row(int H) { return pad4(H) | 4; }
 struct TalkDecodeSmem {                  // float offsets; the staged rows follow at `rows`
   int q, talk, sc, mx, acc, ml, xch, xml, wr, rows, dimp, hp, per, slot;
   __host__ __device__ TalkDecodeSmem(const nb_talk_decode_args& a, int S, int stage) {
-    dimp = (a.dim + 15) & ~15;
+    dimp = ((a.dim + 15) & ~15) + 8;     // rows of neighbouring heads start in different banks
     hp = head_row(a.H);
     per = pad4((a.H * a.vdim + S - 1) / S);
     slot = per;
@@ -508,6 +508,9 @@ struct TalkDecodeSmem {                  // float offsets; the staged rows follo
     rows = wr + (S + 1) * hp;
   }
 };
+
+// i / n for small non-negative numbers
+__device__ __forceinline__ int small_div(int i, int n) { return (int)__fdividef((float)i + 0.5f, (float)n); }
 
 template <typename T> __device__ __forceinline__ int row_pad(int ldc) {      // 16-byte units of a staged row: odd
   return (ldc * (int)sizeof(T) / 16) | 1;
@@ -618,60 +621,53 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     if (mine >= base && mine < base + nk) put_row(rows + (size_t)(mine - base) * ldr);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const int chunks = (rep + 3) / 4, tiles16 = (rep + 15) / 16;
+    const int chunks = (rep + 3) / 4, tiles8 = (rep + 7) / 8;
     auto put_score = [&](int j, int h, float x) {                  // over the penalty that waits there
       float* s = sc + j * hp + h;
       *s = (p.softcap > 0.f ? p.softcap * tanhf(x * isc) : x * isc) - *s;
     };
-    const int ra = lane >> 2, c2 = (lane & 3) * 2;                 // this lane's first row (head) and column pair of a product
+    const int ra = lane >> 2, c2 = (lane & 3) * 2;                 // of a product's fragments: this lane's row, its column pair
     if (mma) {
-      // raw scores on the tensor cores: up to 16 heads of a group x 16 keys per warp; the queries enter as three bf16 terms (a score's
-      // error is an exponent's)
-      const int kt = (nk + 15) / 16;
-      for (int i = warp; i < p.G * tiles16 * kt; i += kTdWarps) {
-        const int gc = i / kt, j0 = (i - gc * kt) * 16, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
-        const bf16* kr = reinterpret_cast<const bf16*>(rows) + (size_t)min(j0 + (lane & 7) + ((lane >> 4) << 3), nk - 1) * ldr + g * D + ((lane >> 3) & 1) * 8;
-        float c[3][2][4] = {};           // a chain of products per term
+      // raw scores on the tensor cores: 16 keys x up to eight heads of a group per warp; the queries enter as three bf16
+      // terms (a score's error is an exponent's)
+      const int kt = (nk + 15) >> 4;
+      for (int i = warp; i < p.G * tiles8 * kt; i += kTdWarps) {
+        const int gc = small_div(i, kt), j0 = (i - gc * kt) * 16, g = small_div(gc, tiles8), hb = g * rep + (gc - g * tiles8) * 8;
+        const int hn = min(8, (g + 1) * rep - hb);
+        const bf16* kr = reinterpret_cast<const bf16*>(rows) + (size_t)min(j0 + (lane & 15), nk - 1) * ldr + g * D + (lane >> 4) * 8;
+        const float* qr = qs + (hb + min(ra, hn - 1)) * L.dimp + c2;               // heads past the group's: not kept
+        float c[3][4] = {};              // a chain of products per term
 #pragma unroll 4
         for (int kk = 0; kk < D; kk += 16) {
-          uint32_t q1[4], q2[4], q3[4], bb[4];
-          ldsm_x4(bb, kr + kk);
+          uint32_t a[4], q1[2], q2[2], q3[2];
+          ldsm_x4(a, kr + kk);
 #pragma unroll
-          for (int f = 0; f < 4; ++f) {
-            const int r = ra + (f & 1) * 8;
-            const float2 v = r < hn ? *reinterpret_cast<const float2*>(qs + (hb + r) * L.dimp + kk + (f >> 1) * 8 + c2) : make_float2(0.f, 0.f);
+          for (int f = 0; f < 2; ++f) {
+            const float2 v = *reinterpret_cast<const float2*>(qr + kk + f * 8);
             split_bf16(v.x, v.y, q1[f], q2[f]);
             q3[f] = pack_bf16(v.x - bf_lo(q1[f]) - bf_lo(q2[f]), v.y - bf_hi(q1[f]) - bf_hi(q2[f]));
           }
-          mma_bf16(c[0][0], q1, bb[0], bb[1]);
-          mma_bf16(c[0][1], q1, bb[2], bb[3]);
-          mma_bf16(c[1][0], q2, bb[0], bb[1]);
-          mma_bf16(c[1][1], q2, bb[2], bb[3]);
-          mma_bf16(c[2][0], q3, bb[0], bb[1]);
-          mma_bf16(c[2][1], q3, bb[2], bb[3]);
+          mma_bf16(c[0], a, q1[0], q1[1]);
+          mma_bf16(c[1], a, q2[0], q2[1]);
+          mma_bf16(c[2], a, q3[0], q3[1]);
+        }
+        float v[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = ((c[2][e] + c[1][e]) + c[0][e]) * isc;
+          // cap tanh(x) = cap - 2 cap / (1 + e^2x): an absolute error of the cap's rounding
+          v[e] = p.softcap > 0.f ? p.softcap - 2.f * p.softcap / (1.f + expf(2.f * x)) : x;
         }
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          if (half * 8 >= hn) break;
-          const int r = ra + half * 8;
-          float v[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const float x = ((c[2][e >> 1][2 * half + (e & 1)] + c[1][e >> 1][2 * half + (e & 1)]) + c[0][e >> 1][2 * half + (e & 1)]) * isc;
-            // cap tanh(x) = cap - 2 cap / (1 + e^2x): an absolute error of the cap's rounding
-            v[e] = p.softcap > 0.f ? p.softcap - 2.f * p.softcap / (1.f + expf(2.f * x)) : x;
-          }
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int j = j0 + (e >> 1) * 8 + c2 + (e & 1);
-            if (j < nk && r < hn) sc[j * hp + hb + r] = v[e] - sc[j * hp + hb + r];
-          }
+        for (int e = 0; e < 4; ++e) {
+          const int j = j0 + ra + (e >> 1) * 8, h = c2 + (e & 1);
+          if (j < nk && h < hn) sc[j * hp + hb + h] = v[e] - sc[j * hp + hb + h];
         }
       }
     } else {
       // a thread takes one key of one group (and up to four of its heads at a time)
       for (int i = tid; i < nk * p.G * chunks; i += kTdThreads) {
-        const int gc = i / nk, j = i - gc * nk, g = gc / chunks, h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
+        const int gc = small_div(i, nk), j = i - gc * nk, g = small_div(gc, chunks), h0 = g * rep + (gc - g * chunks) * 4, hn = min(4, (g + 1) * rep - h0);
         const T* kr = rows + (size_t)j * ldr + g * D;
         const float* qh = qs + h0 * L.dimp;
         float x[4] = {0.f, 0.f, 0.f, 0.f};
@@ -704,16 +700,20 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     for (int h = warp; h < H; h += kTdWarps) {
       const float *t = talk_s + h * hp, old = ml[h];
       float m = old;
-      for (int j = lane; j < nk; j += 32) {
-        const float* s = sc + j * hp;
-        float v = 0.f;
+      for (int j = lane; j < nk; j += 64) {
+        const bool two = j + 32 < nk;
+        const float *s = sc + j * hp, *s2 = s + (two ? 32 * hp : 0);
+        float v = 0.f, v2 = 0.f;
 #pragma unroll 4
         for (int g = 0; g < hp; g += 4) {
           const float4 a = *reinterpret_cast<const float4*>(t + g), c = *reinterpret_cast<const float4*>(s + g);
+          const float4 d = *reinterpret_cast<const float4*>(s2 + g);
           v += (a.x * c.x + a.y * c.y) + (a.z * c.z + a.w * c.w);
+          v2 += (a.x * d.x + a.y * d.y) + (a.z * d.z + a.w * d.w);
         }
         mx[j * hp + h] = v;
-        m = fmaxf(m, v);
+        if (two) mx[(j + 32) * hp + h] = v2;
+        m = fmaxf(m, fmaxf(v, v2));
       }
       m = warp_max(m);
       float sum = 0.f;
@@ -732,51 +732,46 @@ __global__ void __launch_bounds__(kTdThreads, 1) talk_decode_kernel(const nb_tal
     }
     __syncthreads();
     if (mma) {
-      // weighted values: up to 16 heads of a group x up to kCt tiles of 16 columns per warp; the weights enter as two bf16 terms
+      // weighted values: up to kCt tiles of 16 columns x up to eight heads of a group per warp; the weights enter as two bf16
+      // terms
       constexpr int kCt = 4;
-      const int ct = (V + 15) / 16, tpw = min(kCt, (p.G * tiles16 * ct + kTdWarps - 1) / kTdWarps), parts = (ct + tpw - 1) / tpw;
-      for (int i = warp; i < p.G * tiles16 * parts; i += kTdWarps) {
-        const int gc = i / parts, t0 = (i - gc * parts) * tpw, g = gc / tiles16, hb = g * rep + (gc - g * tiles16) * 16, hn = min(16, (g + 1) * rep - hb);
-        const int tn = min(tpw, ct - t0);
-        const bf16* vr = reinterpret_cast<const bf16*>(rows) + p.v_off + g * V + t0 * 16 + (lane >> 4) * 8;
-        float c[kCt][2][4] = {};
+      const int ct = (V + 15) >> 4, tpw = min(kCt, (p.G * tiles8 * ct + kTdWarps - 1) / kTdWarps), parts = small_div(ct + tpw - 1, tpw);
+      for (int i = warp; i < p.G * tiles8 * parts; i += kTdWarps) {
+        const int gc = small_div(i, parts), t0 = (i - gc * parts) * tpw, g = small_div(gc, tiles8), hb = g * rep + (gc - g * tiles8) * 8;
+        const int hn = min(8, (g + 1) * rep - hb), tn = min(tpw, ct - t0);
+        // the values' tile, transposed: columns are the product's rows, keys its depth
+        const bf16* vr = reinterpret_cast<const bf16*>(rows) + p.v_off + g * V + t0 * 16 + ((lane >> 3) & 1) * 8;
+        const float* w = mx + hb + min(ra, hn - 1);                                // heads past the group's: not kept
+        float c[kCt][2][4] = {};         // a chain of products per term
 #pragma unroll 2
         for (int kk = 0; kk < nk; kk += 16) {
-          uint32_t hi[4], lo[4];
+          uint32_t hi[2], lo[2];
 #pragma unroll
-          for (int f = 0; f < 4; ++f) {
-            const int r = ra + (f & 1) * 8, j = kk + (f >> 1) * 8 + c2;
-            const float* w = mx + j * hp + hb + r;
-            split_bf16(r < hn && j < nk ? w[0] : 0.f, r < hn && j + 1 < nk ? w[hp] : 0.f, hi[f], lo[f]);
+          for (int f = 0; f < 2; ++f) {
+            const int j = kk + f * 8 + c2;                                         // keys past the stage have no weight
+            split_bf16(j < nk ? w[j * hp] : 0.f, j + 1 < nk ? w[(j + 1) * hp] : 0.f, hi[f], lo[f]);
           }
-          const bf16* vk = vr + (size_t)min(kk + (lane & 15), nk - 1) * ldr;       // keys past the stage have no weight
-          uint32_t bb[kCt][4];
+          const bf16* vk = vr + (size_t)min(kk + (lane & 7) + ((lane >> 4) << 3), nk - 1) * ldr;
 #pragma unroll
           for (int y = 0; y < kCt; ++y)
-            if (y < tn) ldsm_x4_t(bb[y], vk + y * 16);
-#pragma unroll
-          for (int term = 0; term < 2; ++term)
-#pragma unroll
-            for (int y = 0; y < kCt; ++y)
-              if (y < tn) {
-                mma_bf16(c[y][0], term ? lo : hi, bb[y][0], bb[y][1]);
-                mma_bf16(c[y][1], term ? lo : hi, bb[y][2], bb[y][3]);
-              }
+            if (y < tn) {
+              uint32_t a[4];
+              ldsm_x4_t(a, vk + y * 16);
+              mma_bf16(c[y][0], a, hi[0], hi[1]);
+              mma_bf16(c[y][1], a, lo[0], lo[1]);
+            }
         }
 #pragma unroll
         for (int y = 0; y < kCt; ++y)
           if (y < tn) {
 #pragma unroll
-            for (int x = 0; x < 2; ++x)
-#pragma unroll
-              for (int half = 0; half < 2; ++half) {
-                const int v = (t0 + y) * 16 + x * 8 + c2, r = ra + half * 8;       // V is a multiple of 8
-                if (v < V && r < hn) {
-                  float2* a = reinterpret_cast<float2*>(acc + (hb + r) * V + v);
-                  const float f = wr[hb + r];
-                  *a = make_float2(fmaf(a->x, f, c[y][x][2 * half]), fmaf(a->y, f, c[y][x][2 * half + 1]));
-                }
+            for (int e = 0; e < 4; ++e) {
+              const int v = (t0 + y) * 16 + ra + (e >> 1) * 8, h = c2 + (e & 1);
+              if (v < V && h < hn) {
+                float* a = acc + (hb + h) * V + v;
+                *a = fmaf(*a, wr[hb + h], c[y][0][e] + c[y][1][e]);
               }
+            }
           }
       }
     } else {
