@@ -1,5 +1,6 @@
 /* nativebit_b200 — C ABI of the kernels of layered decoders (models that list their layers one by one: latent
- * attention, gated linear attention, dense feed-forward, norms before and after every sublayer).
+ * attention, grouped attention with scores mixed across heads, gated linear attention, dense feed-forward, norms before and
+ * after every sublayer or hyper-connections).
  *
  * Same rules as nativebit_b200.h: plain device pointers, sizes and a CUDA stream handle; asynchronous; no
  * allocation, no synchronisation; every call returns an nb_status; no CPU path.  Weights are bf16, row-major

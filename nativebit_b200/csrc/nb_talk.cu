@@ -270,8 +270,8 @@ __global__ void __launch_bounds__(kPvThreads, VD <= 128 ? 3 : 1) talk_values_bf1
   extern __shared__ __align__(16) bf16 v_s[];   // [2][64][VD + 8]
   constexpr int vp = VD + 8;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int h = blockIdx.y / vtiles, v0 = (blockIdx.y - h * vtiles) * VD, vn = min(VD, p.vdim - v0), b = blockIdx.z;
-  const int tile = blk.tile0 + blockIdx.x, q0 = tile * kQT;
+  const int h = blockIdx.x / vtiles, v0 = (blockIdx.x - h * vtiles) * VD, vn = min(VD, p.vdim - v0), b = blockIdx.z;
+  const int local = gridDim.y - 1 - blockIdx.y, q0 = (blk.tile0 + local) * kQT;    // longest first
   const int first = talk_first_key(p.pos0, q0, p.window), last = p.pos0 + min(q0 + kQT - 1, p.T - 1), tiles = (last - first) / kKT + 1;
   const bf16* vals = reinterpret_cast<const bf16*>(p.cache) + (size_t)b * p.ctx * p.ldc + p.v_off + (h / (p.H / p.G)) * p.vdim + v0;
   for (int i = tid; i < 2 * kKT * (vp - vn); i += kPvThreads) {    // columns past the values stay zero
@@ -302,7 +302,7 @@ __global__ void __launch_bounds__(kPvThreads, VD <= 128 ? 3 : 1) talk_values_bf1
   };
   copy_tile(0, 0);
   const int rowa = warp * 16 + (lane >> 2), c2 = (lane & 3) * 2;
-  const float* ws = blk.ws + (((size_t)(b * blk.tiles + blockIdx.x) * p.H + h) * kQT + rowa) * blk.ld + c2;
+  const float* ws = blk.ws + (((size_t)(b * blk.tiles + local) * p.H + h) * kQT + rowa) * blk.ld + c2;
   const size_t row8 = (size_t)8 * blk.ld;
   float2 nx[8][2];                       // the next tile's scores: rows a and b, eight pairs of keys
   auto load_scores = [&](int t) {
@@ -912,7 +912,7 @@ template <int VD> static int launch_values_bf16(const nb_talk_attention_args& a,
   }
   const int vec = a.vdim % 8 == 0 && a.ldc % 8 == 0 && a.v_off % 8 == 0 && a.ldo % 2 == 0 && a.ldg % 2 == 0 && (uintptr_t)a.cache % 16 == 0 &&
                   (uintptr_t)a.out % 4 == 0 && (uintptr_t)a.gate % 4 == 0;
-  talk_values_bf16_kernel<VD><<<dim3(blk.tiles, a.H * vtiles, a.B), kPvThreads, smem, st>>>(a, blk, vtiles, vec);
+  talk_values_bf16_kernel<VD><<<dim3(a.H * vtiles, blk.tiles, a.B), kPvThreads, smem, st>>>(a, blk, vtiles, vec);
   return check_launch();
 }
 

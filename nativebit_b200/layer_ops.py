@@ -181,7 +181,7 @@ def cache_append(src: torch.Tensor, offset: int, cols: int, cache: torch.Tensor,
           cache.shape[1], pos0, _stream())
 
 
-TALK_WORKSPACE = 384 << 20             # bytes of mixed scores at a time: fewer, longer launches measured faster than a block that stays in L2
+TALK_WORKSPACE = 256 << 20             # bytes of mixed scores at a time: fewer, longer launches measured faster than a block that stays in L2
 
 
 def talk_workspace_bytes(b: int, t: int, heads: int, pos0: int, window: int, tiles: int) -> int:
