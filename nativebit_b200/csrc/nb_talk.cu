@@ -873,7 +873,7 @@ template <int HM, int NB, bool kTwo> static int launch_scores_mma(const nb_talk_
   }
   const int vec = a.dim % 8 == 0 && a.ldq % 8 == 0 && a.ldc % 8 == 0 && (uintptr_t)a.q % 16 == 0 && (uintptr_t)a.cache % 16 == 0;
   const int steps = (blk.ld + 64 * NB - 1) / (64 * NB), subs = blk.tiles * (kQT / kSq);
-  const int chunk = std::max(1, std::min(steps, (int)((long long)steps * subs * a.B / (4 * sm_count()))));   // about four CTAs per SM
+  const int chunk = std::max(1, std::min(steps, (int)((long long)steps * subs * a.B / (2 * sm_count()))));   // about two CTAs per SM, one after the other
   talk_scores_bf16_kernel<HM, NB, kTwo><<<dim3((steps + chunk - 1) / chunk, subs, a.B), kScThreads, talk_scores_smem(a, HM, NB, stages), st>>>(
       a, blk, (a.dim + 15) & ~15, chunk, stages, vec);
   return check_launch();

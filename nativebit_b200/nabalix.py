@@ -67,7 +67,9 @@ def build(config: dict, tensor, dtype: torch.dtype, context_len: int) -> Layered
 
 
 def load(folder: str, config: dict, dtype: torch.dtype, context_len: int, device) -> LayeredDecoder:
-    return load_checkpoint(folder, device, lambda tensor: build(config, tensor, dtype, context_len))
+    # a layer without a feed-forward may carry the connection of one
+    spare = tuple(f"l{i}.{n}" for i, spec in enumerate(config["layers"]) if spec["mlp"] is None for n in ("norm2", "ls2", "hc2."))
+    return load_checkpoint(folder, device, lambda tensor: build(config, tensor, dtype, context_len), spare)
 
 
 def random_tensors(config: dict, seed: int, device) -> dict[str, torch.Tensor]:

@@ -51,12 +51,14 @@ class Checkpoint:
         return sorted(set(self._index) - self._read)
 
 
-def load_checkpoint(folder: str, device, build):
-    """build(tensor) with tensor(name, shape) -> the weight on the device; every tensor of the file must be asked for."""
+def load_checkpoint(folder: str, device, build, spare: tuple = ()):
+    """build(tensor) with tensor(name, shape) -> the weight on the device; every tensor of the file must be asked for, except
+    those whose names begin with one of `spare`."""
     ckpt = Checkpoint(f"{folder}/model.safetensors", device)
     model = build(lambda n, s: ckpt.get(n, s))
-    if ckpt.unread():
-        raise ValueError(f"the checkpoint has tensors that the configuration does not name: {ckpt.unread()[:8]}")
+    unknown = [n for n in ckpt.unread() if not n.startswith(spare)] if spare else ckpt.unread()
+    if unknown:
+        raise ValueError(f"the checkpoint has tensors that the configuration does not name: {unknown[:8]}")
     torch.cuda.synchronize(device)           # the kernels request weights before they wait for earlier work of the stream
     return model
 

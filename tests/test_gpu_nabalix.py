@@ -559,8 +559,11 @@ def test_unknown_tensors_are_refused(dev, tmp_path):
     from nativebit_b200 import registry
     from nativebit_b200.weights import write_safetensors
     w = nc.weights(nc.CASES["mixed"], seed=5)
-    w["l0.mix.extra"] = torch.zeros(4, 4).bfloat16()
     (tmp_path / "config.json").write_text(json.dumps(nc.CASES["mixed"]))
-    write_safetensors(str(tmp_path / "model.safetensors"), w)
-    with pytest.raises(ValueError):
-        registry.load_model(str(tmp_path), "float32", 64)
+    for extra, known in (("l1.norm2", True), ("l1.hc2.in", True), ("l0.mix.extra", False)):      # layer 1 has no feed-forward
+        write_safetensors(str(tmp_path / "model.safetensors"), {**w, extra: torch.zeros(3).bfloat16()})
+        if known:
+            registry.load_model(str(tmp_path), "float32", 64)
+        else:
+            with pytest.raises(ValueError):
+                registry.load_model(str(tmp_path), "float32", 64)
