@@ -204,6 +204,50 @@ def test_talk_attention(dev, shape, dtype, T, pos0, window, tiles):
     close(out[:, :H * V], ref, 2e-5 if dtype == F32 else 2.0 ** -7)
 
 
+def dense_attention(q, k, v, scale, cap, r1, r2, talk, window):
+    """O.mixed_head_attention over whole matrices (the oracle's own test holds the two together)."""
+    T, H, _ = q.shape
+    rep = H // k.shape[1]
+    i = np.arange(T)
+    s = np.einsum("ihd,jhd->hij", q, np.repeat(k, rep, 1), optimize=True) * scale
+    far = np.maximum(i[:, None] - i[None], 0)
+    s = cap * np.tanh(s / cap) - r1.astype(np.float64)[:, None, None] * np.log1p(r2.astype(np.float64)[:, None, None] * far)
+    s = np.tensordot(talk.astype(np.float64), s, 1)
+    s[:, (i[None, :] > i[:, None]) | (i[:, None] - i[None, :] >= window)] = -np.inf
+    p = np.exp(s - s.max(-1, keepdims=True))
+    return np.einsum("hij,jhd->ihd", p / p.sum(-1, keepdims=True), np.repeat(v, rep, 1), optimize=True)
+
+
+@pytest.mark.parametrize("shape", [SHAPES[0], SHAPES[2], SHAPES[5], dict(H=10, G=5, D=48, V=32), dict(H=9, G=3, D=40, V=24),
+                                   dict(H=20, G=4, D=160, V=16)])
+@pytest.mark.parametrize("B,T,pos0,window,tiles", [(3, 1400, 30, 700, 99), (1, 330, 100, 290, 2), (3, 1400, 0, 2000, 7)])
+def test_talk_attention_over_many_steps(dev, shape, B, T, pos0, window, tiles):
+    """Windows of many tiles and enough queries that a CTA walks several steps of keys (one sequence, B times)."""
+    from nativebit_b200 import layer_ops as L
+    H, G, D, V = (shape[k] for k in "HGDV")
+    N = pos0 + T
+    q, k, v, talk, r1, r2, gate = attention_inputs(shape, 1, N, BF16, T + D, pos0, max(0, N - window - T // 3))
+    scale, cap = 4.0 / np.sqrt(D), 8.0
+    ref = np.tile(dense_attention(q[0], k[0], v[0], scale, cap, r1, r2, talk, window)[pos0:].reshape(T, H * V), (B, 1))
+    q, k, v, gate = (np.repeat(x, B, 0) for x in (q, k, v, gate))
+    ref = ref * HO.sigmoid(gate[:, pos0:].reshape(B * T, H * V))
+    v_off = L.pad8(G * D)
+    cache = torch.zeros(B, N, v_off + L.pad8(G * V), dtype=BF16, device=dev)
+    cache[:, :, :G * D], cache[:, :, v_off:v_off + G * V] = cu(k.reshape(B, N, G * D), BF16), cu(v.reshape(B, N, G * V), BF16)
+    qt, gt, out = (L.rows_empty(B * T, n, BF16, dev) for n in (H * D, H * V, H * V))
+    qt[:, :H * D], gt[:, :H * V] = cu(q[:, pos0:].reshape(B * T, H * D), BF16), cu(gate[:, pos0:].reshape(B * T, H * V), BF16)
+    n_pen = min(window, N)
+    pen, tk = penalty_table(r1, r2, n_pen), cu(talk)
+    from nativebit_b200 import _lib
+    a = _lib.TalkAttentionArgs(q=qt.data_ptr(), cache=cache.data_ptr(), gate=gt.data_ptr(), out=out.data_ptr(), penalty=pen.data_ptr(),
+                               talk=tk.data_ptr(), scale=scale, softcap=cap, dtype=L._DTYPE[BF16], B=B, T=T, H=H, G=G, dim=D, vdim=V, ctx=N,
+                               ldc=cache.shape[2], v_off=v_off, ldq=qt.stride(0), ldg=gt.stride(0), ldo=out.stride(0), pos0=pos0, window=window,
+                               n_pen=n_pen)
+    ws = torch.full((L.talk_workspace_bytes(B, T, H, pos0, window, tiles),), 255, dtype=torch.uint8, device=dev)
+    L.talk_attention_in(ws, a)
+    close(out[:, :H * V], ref, 2.0 ** -7)
+
+
 def test_talk_attention_without_its_options(dev):
     """No cap, no penalty, no gate, no window, heads not mixed: ordinary grouped attention."""
     from nativebit_b200 import _lib
